@@ -10,7 +10,9 @@
  * window plus kept first tokens and a sink in the denominator; clamped gated dense feed-forward; routed gated experts),
  * and one-norm-per-layer blocks with plain RMS weights whose layers may repeat (gated linear attention, attention inside
  * chunks of positions with a linear distance bias, latent attention with full-rank queries; gated dense feed-forward,
- * routed clamped experts beside identity experts).
+ * routed clamped experts beside identity experts), and norm - sublayer - norm blocks with plain RMS weights (retention,
+ * softmax attention whose values are its unrotated keys beside a gated delta rule with one decay per head, latent attention
+ * inside a window with an output gate; group-limited routed experts beside identity experts).
  *
  * Same conventions as jacobi_b200.h: every function returns 0 or a negative status, hy_last_error(h) gives the text,
  * plain pointers and sizes only, host buffers are caller-owned, device memory belongs to the handle, one host thread per
@@ -35,24 +37,25 @@ typedef struct hy_engine* hy_handle;
 typedef enum { HY_OK = 0, HY_ERR_INVALID = -1, HY_ERR_CUDA = -2, HY_ERR_CAPACITY = -3, HY_ERR_UNSUPPORTED = -4 } hy_status;
 typedef enum { HY_DTYPE_BF16 = 0, HY_DTYPE_F32 = 1, HY_DTYPE_F16 = 2, HY_DTYPE_I32 = 3 } hy_dtype;
 typedef enum { HY_MIX_ATTN_SCAN = 0, HY_MIX_DELTA = 1, HY_MIX_SSD = 2, HY_MIX_LATENT = 3, HY_MIX_GLR = 4, HY_MIX_WINDOW = 5,
-               HY_MIX_MLSTM = 6, HY_MIX_BIASED = 7, HY_MIX_GLA = 8 } hy_mixer_kind;
+               HY_MIX_MLSTM = 6, HY_MIX_BIASED = 7, HY_MIX_GLA = 8, HY_MIX_RETENTION = 9, HY_MIX_ATTN_DELTA = 10 } hy_mixer_kind;
 /* HY_FF_GATED: down(act(gate x) * (up x)), act = hy_act_kind in ff_act */
 typedef enum { HY_FF_NONE = 0, HY_FF_RELU2 = 1, HY_FF_ROUTED = 2, HY_FF_GATED = 3 } hy_ff_kind;
 /* HY_ACT_CLAMPED (gated pairs only, dense or in experts): g = min(gate, limit), u = clamp(up, -limit, limit), g sigmoid(1.702 g) (u + 1) */
 typedef enum { HY_ACT_SILU = 0, HY_ACT_GELU_TANH = 1, HY_ACT_GELU_ERF = 2, HY_ACT_CLAMPED = 3 } hy_act_kind;
 /* how a routed feed-forward scores its experts: sigmoid scores, group-limited choice, weights normalised to x_scale |
  * the largest logits (plus a bias per expert), weights = softmax over the chosen logits alone | softmax scores over all
- * router outputs, choice by score + correction (one number per output), weights = the chosen scores as they are */
+ * router outputs, choice by score + correction (one number per output) inside the x_keep groups of neighbouring outputs with
+ * the largest single choice scores, weights = the chosen scores as they are */
 typedef enum { HY_ROUTE_SIGMOID_GROUPS = 0, HY_ROUTE_TOP_SOFTMAX = 1, HY_ROUTE_CORRECTED_SOFTMAX = 2 } hy_route_kind;
 /* what the distance takes off a score of HY_MIX_BIASED: r1_h ln(1 + r2_h (i - j)) with learned r1, r2 |
- * 2^(-8 (h + 1) / heads) (i - j), no tensors */
-typedef enum { HY_BIAS_LOG = 0, HY_BIAS_LINEAR = 1 } hy_bias_kind;
+ * 2^(-8 (h + 1) / heads) (i - j), no tensors | nothing */
+typedef enum { HY_BIAS_LOG = 0, HY_BIAS_LINEAR = 1, HY_BIAS_NONE = 2 } hy_bias_kind;
 /* norm of the residual stream: RMS with a weight stored as an offset from one | tanh(alpha x) w + b (no statistics) |
  * RMS with a plain weight */
 typedef enum { HY_NORM_RMS_OFFSET = 0, HY_NORM_TANH = 1, HY_NORM_RMS = 2 } hy_norm_kind;
 /* HY_BLOCK_PARALLEL: x += mixer(n(x)) + ff(n(x)), one norm per layer (HY_NORM_RMS_OFFSET or HY_NORM_RMS).
  * HY_BLOCK_SANDWICH: x += ls1 * n1b(mixer(n1(x))), then x += ls2 * n2b(ff(n2(x))): a norm on both sides of each sublayer
- * and a per-channel layer scale.
+ * and a per-channel layer scale (HY_NORM_TANH), or no layer scale (HY_NORM_RMS).
  * HY_BLOCK_POSTNORM: x += ls1 * n1(mixer(x)), then x += ls2 * n2(ff(x)): the sublayers read the stream itself, the norm
  * (RMS, with statistics over the width) sits on the sublayer's output.
  * HY_BLOCK_PRENORM: x += m ls1 mixer(c1(n1(x))), then x += m ls2 ff(c2(n2(x))): RMS norms with plain weights on the
@@ -126,6 +129,15 @@ typedef struct {
   float g_tau;
   /* more of HY_FF_ROUTED: router outputs behind the experts that stand for the input itself */
   int32_t x_identity;
+  /* more of HY_MIX_LATENT: position i sees j with 0 <= i - j < l_window only (0: every j <= i); 1 = the concatenated heads are
+   * multiplied by sigmoid of a gate projection ("g"), element by element */
+  int32_t l_window, l_gate;
+  /* HY_MIX_RETENTION (linear attention with one fixed decay per head): sizes in g_heads, g_dim, g_vdim, rotation of queries
+   * and keys in r_*; the decays come as the fp32 tensor "l<i>.mix.decay" [heads], which the host makes of its configuration.
+   * HY_MIX_ATTN_DELTA (two mixers on one input): softmax attention whose values are its keys before their rotation and whose
+   * heads have one output gate each, tensors "mix.left.*", sizes in b_heads, b_kv_heads, b_dim = b_vdim, b_scale, rotation in
+   * r_*; gated delta rule with one decay per head and a silu output gate, tensors "mix.right.*", sizes in d_*; summed with
+   * left_scale and right_scale */
 } hy_layer_cfg;
 
 typedef struct {

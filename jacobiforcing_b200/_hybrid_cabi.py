@@ -10,7 +10,7 @@ import subprocess
 _HERE = os.path.dirname(os.path.abspath(__file__))
 ROOT = os.path.dirname(_HERE)
 LIB_PATH = os.path.join(_HERE, "libjf_hybrid.so")
-SOURCES = [os.path.join(_HERE, "csrc", f) for f in ("hy_engine.cu", "hy_kernels.cuh", "hy_gemm.cuh", "hy_attn.cuh", "hy_mixers.cuh", "hy_experts.cuh", "hy_window.cuh", "hy_biased.cuh", "hy_gla.cuh",
+SOURCES = [os.path.join(_HERE, "csrc", f) for f in ("hy_engine.cu", "hy_kernels.cuh", "hy_gemm.cuh", "hy_attn.cuh", "hy_mixers.cuh", "hy_experts.cuh", "hy_window.cuh", "hy_biased.cuh", "hy_gla.cuh", "hy_delta.cuh",
                                                         "jf_ptx.cuh")] + [
     os.path.join(ROOT, "include", "jacobi_hybrid.h")]
 NVCC_FLAGS = ["-gencode", "arch=compute_100a,code=sm_100a", "-O3", "-lineinfo", "-std=c++17", "-shared", "-Xcompiler", "-fPIC"]
@@ -43,7 +43,7 @@ class LayerCfg(C.Structure):
                 [(n, C.c_int32) for n in ("b_heads", "b_kv_heads", "b_dim", "b_vdim", "b_window", "b_keep_first", "b_v_mix")] +
                 [("b_scale", C.c_float), ("b_softcap", C.c_float), ("ff_limit", C.c_float)] +
                 [(n, C.c_int32) for n in ("l_no_sink", "r_half", "b_chunk", "b_bias", "b_unit_sink", "b_qk_norm", "b_no_bias", "g_low")] +
-                [("g_tau", C.c_float), ("x_identity", C.c_int32)])
+                [("g_tau", C.c_float), ("x_identity", C.c_int32), ("l_window", C.c_int32), ("l_gate", C.c_int32)])
 
 
 class ModelCfg(C.Structure):

@@ -10,6 +10,8 @@
 // and leaves unnormalised partial results (m, l, O) per (row, split).  The combine kernel merges the splits of a row with
 // the sink (a logit with no key and no value: it only enters the maximum and the denominator), applies the output gate
 // and the mixer's scale and writes the operand of the output projection.
+// Key splits are runs of split_keys absolute positions, counted per tile from the one that holds the first position its first
+// row sees: with a sliding window a tile has no units for the keys before its window (see first_split).
 #pragma once
 #include "hy_kernels.cuh"
 #include "jf_ptx.cuh"
@@ -18,10 +20,13 @@ namespace hy {
 
 struct AttnUnit { int entry, kv_head, row0, split; };   // row0: first row of the tile inside the entry (rows = tokens x R)
 
+// absolute index of a tile's first key split; p: position of the tile's first row
+__host__ __device__ __forceinline__ int first_split(int p, int window, int split_keys) { return first_seen(p, window) / split_keys; }
+
 template <int DIM>
 __global__ void __launch_bounds__(128) attn_mma_kernel(Batch b, const AttnUnit* __restrict__ units, const bf16* __restrict__ q,
                                                        int ldq, const bf16* __restrict__ cache, int H, int G, float scale,
-                                                       float qt_coef, int qt_every, int split_keys, int n_splits, int vdim,
+                                                       float qt_coef, int qt_every, int window, int split_keys, int n_splits, int vdim,
                                                        float* __restrict__ part_o, float* __restrict__ part_ml) {
   constexpr int LD = DIM + 8;                           // padded row (elements): ldmatrix rows fall into distinct banks
   __shared__ __align__(16) bf16 qs[64 * LD];
@@ -62,8 +67,10 @@ __global__ void __launch_bounds__(128) attn_mma_kernel(Batch b, const AttnUnit* 
   for (int i = 0; i < DIM / 8; ++i) { o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.0f; }
   // key range of this unit: its split, cut at the last position any row of the tile may see
   const int last_row = min(u.row0 + 63, rows_total - 1);
-  const int key_end = min((u.split + 1) * split_keys, pos0 + last_row / R + 1);
-  for (int j0 = u.split * split_keys; j0 < key_end; j0 += 64) {
+  const int p_tile = pos0 + u.row0 / R, split = first_split(p_tile, window, split_keys) + u.split;
+  const int key_end = min((split + 1) * split_keys, pos0 + last_row / R + 1);
+  const int f_lo_key = first_seen(max(p_lo, 0), window), f_hi_key = first_seen(max(p_hi, 0), window);
+  for (int j0 = max(split * split_keys, first_seen(p_tile, window) / 64 * 64); j0 < key_end; j0 += 64) {
     __syncthreads();                                     // the previous tile has been read
     for (int i = tid; i < 64 * (DIM / 8); i += 128) {
       const int r = i / (DIM / 8), c = i % (DIM / 8);
@@ -99,8 +106,8 @@ __global__ void __launch_bounds__(128) attn_mma_kernel(Batch b, const AttnUnit* 
 #pragma unroll
       for (int c = 0; c < 2; ++c) {
         const int j = j0 + nb * 8 + (lane & 3) * 2 + c;
-        s[nb][c] = (j <= p_lo && j < key_end) ? s[nb][c] * f_lo : -INFINITY;
-        s[nb][2 + c] = (j <= p_hi && j < key_end) ? s[nb][2 + c] * f_hi : -INFINITY;
+        s[nb][c] = (j <= p_lo && j >= f_lo_key && j < key_end) ? s[nb][c] * f_lo : -INFINITY;
+        s[nb][2 + c] = (j <= p_hi && j >= f_hi_key && j < key_end) ? s[nb][2 + c] * f_hi : -INFINITY;
         mx_lo = fmaxf(mx_lo, s[nb][c]);
         mx_hi = fmaxf(mx_hi, s[nb][2 + c]);
       }
@@ -193,7 +200,7 @@ __global__ void __launch_bounds__(128) attn_mma_kernel(Batch b, const AttnUnit* 
 template <int NT>
 __global__ void __launch_bounds__(256, 1) attn_wide_kernel(Batch b, const AttnUnit* __restrict__ units, const bf16* __restrict__ q,
                                                            int ldq, const bf16* __restrict__ cache, int H, int dk, int vdim,
-                                                           float scale, int split_keys, int n_splits, int pstride,
+                                                           float scale, int window, int split_keys, int n_splits, int pstride,
                                                            float* __restrict__ part_o, float* __restrict__ part_ml) {
   extern __shared__ __align__(16) unsigned char hy_smem[];
   const int dkp = (dk + 15) & ~15, LD = dkp + 8;          // padded row (elements): ldmatrix rows fall into distinct banks
@@ -241,9 +248,11 @@ __global__ void __launch_bounds__(256, 1) attn_wide_kernel(Batch b, const AttnUn
 #pragma unroll
     for (int nt = 0; nt < NT; ++nt) { o[mt][nt][0] = o[mt][nt][1] = o[mt][nt][2] = o[mt][nt][3] = 0.0f; }
   const int last_row = min(u.row0 + 63, rows_total - 1);
-  const int key_end = min((u.split + 1) * split_keys, pos0 + last_row / H + 1);
+  const int p_tile = pos0 + u.row0 / H, split = first_split(p_tile, window, split_keys) + u.split;
+  const int key_end = min((split + 1) * split_keys, pos0 + last_row / H + 1);
+  const int f_lo = first_seen(max(p_lo, 0), window), f_hi = first_seen(max(p_hi, 0), window);
   const int d0 = warp * NT * 8;                           // this warp's value dimensions
-  for (int j0 = u.split * split_keys; j0 < key_end; j0 += 64) {
+  for (int j0 = max(split * split_keys, first_seen(p_tile, window) / 64 * 64); j0 < key_end; j0 += 64) {
     __syncthreads();                                      // the previous tile (keys and weights) has been read
     for (int i = tid; i < 64 * chunks; i += 256) {
       const int r = i / chunks, c = i % chunks;
@@ -281,8 +290,8 @@ __global__ void __launch_bounds__(256, 1) attn_wide_kernel(Batch b, const AttnUn
 #pragma unroll
       for (int c = 0; c < 2; ++c) {
         const int j = j0 + sk0 + nb * 8 + (lane & 3) * 2 + c;
-        s[nb][c] = (j <= p_lo && j < key_end) ? s[nb][c] * scale : -INFINITY;
-        s[nb][2 + c] = (j <= p_hi && j < key_end) ? s[nb][2 + c] * scale : -INFINITY;
+        s[nb][c] = (j <= p_lo && j >= f_lo && j < key_end) ? s[nb][c] * scale : -INFINITY;
+        s[nb][2 + c] = (j <= p_hi && j >= f_hi && j < key_end) ? s[nb][2 + c] * scale : -INFINITY;
         mx_lo = fmaxf(mx_lo, s[nb][c]);
         mx_hi = fmaxf(mx_hi, s[nb][2 + c]);
       }
@@ -393,23 +402,30 @@ constexpr size_t attn_wide_smem(int dk) {
 }
 
 // Merge the key splits of one (token, head) with the sink, gate the result, scale it, write the projection's operand.
-// part_o rows are dim wide; the first vdim of them are values.
+// part_o rows are dim wide; the first vdim of them are values.  G: key heads (a row's tile is found from it).
 template <typename WT, typename OT>
 __global__ void attn_combine_kernel(Batch b, const float* __restrict__ part_o, const float* __restrict__ part_ml,
-                                    const WT* __restrict__ sink, const bf16* __restrict__ gate, int ldg, int H, int dim,
-                                    int vdim, int split_keys, int n_splits, float out_scale, OT* __restrict__ out, int ldo) {
+                                    const WT* __restrict__ sink, const bf16* __restrict__ gate, int ldg, int H, int G, int dim,
+                                    int vdim, int window, int split_keys, int n_splits, float out_scale, OT* __restrict__ out, int ldo) {
   const int t = blockIdx.x / H, h = blockIdx.x % H;
-  const int live = b.tok_pos[t] / split_keys + 1;          // splits that hold a key this row may see
+  int from = 0, live = b.tok_pos[t] / split_keys + 1;      // splits that hold a key this row may see
+  if (window > 0) {
+    const int e = b.tok_ent[t], R = H / G;
+    const int row0 = ((t - b.ent_start[e]) * R + h % R) / 64 * 64;
+    const int tile = first_split(b.ent_pos0[e] + row0 / R, window, split_keys);
+    from = first_split(b.tok_pos[t], window, split_keys) - tile;
+    live -= tile;
+  }
   const float sk = sink ? to_f(sink[h]) : -INFINITY;       // sink NULL: an ordinary softmax
   const size_t slot0 = ((size_t)t * H + h) * n_splits;
   float M = sk;
-  for (int s = 0; s < live; ++s) M = fmaxf(M, part_ml[(slot0 + s) * 2]);
+  for (int s = from; s < live; ++s) M = fmaxf(M, part_ml[(slot0 + s) * 2]);
   float L = expf(sk - M);
-  for (int s = 0; s < live; ++s) L += part_ml[(slot0 + s) * 2 + 1] * expf(part_ml[(slot0 + s) * 2] - M);
+  for (int s = from; s < live; ++s) L += part_ml[(slot0 + s) * 2 + 1] * expf(part_ml[(slot0 + s) * 2] - M);
   const float inv = 1.0f / L;
   for (int d = threadIdx.x; d < vdim; d += blockDim.x) {
     float acc = 0.0f;
-    for (int s = 0; s < live; ++s) acc += part_o[(slot0 + s) * dim + d] * expf(part_ml[(slot0 + s) * 2] - M);
+    for (int s = from; s < live; ++s) acc += part_o[(slot0 + s) * dim + d] * expf(part_ml[(slot0 + s) * 2] - M);
     const float gt = gate ? sigmoid_f(to_f(gate[(size_t)t * ldg + h * vdim + d])) : 1.0f;
     out[(size_t)t * ldo + h * vdim + d] = from_f<OT>(acc * inv * gt * out_scale);
   }

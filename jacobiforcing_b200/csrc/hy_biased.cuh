@@ -25,8 +25,10 @@ namespace hy {
 struct BiasedCfg {
   int H, G, dim, vdim, window, keep;
   float scale, cap;
-  const float* r1; const float* r2; const float* sink;       // [H] each, fp32 (r2 unused by a linear bias)
-  int chunk, linear;
+  const float* r1; const float* r2; const float* sink;       // [H] each, fp32 (r2 unused by a linear bias; sink NULL: ordinary softmax)
+  int chunk, bias;                                           // bias: hy_bias_kind (0 logarithmic, 1 linear, 2 none: r1, r2 unused)
+  const float* gate; int ldg; float out_scale;               // gate [T, ldg] fp32 (NULL: none): head h's output times sigmoid(gate[t, h]) * out_scale
+  __device__ __forceinline__ float out_factor(int t, int h) const { return gate ? sigmoid_f(gate[(size_t)t * ldg + h]) * out_scale : out_scale; }
   // first position of the window or chunk of position p
   __host__ __device__ int first(int p) const {
     if (chunk > 0) return p / chunk * chunk;
@@ -279,8 +281,8 @@ __global__ void __launch_bounds__(128) biased_attn_kernel(Batch b, const AT* __r
   const int w0 = c.first(pos);                                                      // first token of the window or chunk
   const int nk = min(c.keep, w0);                                                   // kept first tokens outside the window
   const int n = nk + pos + 1 - w0;
-  const float r1 = c.r1[h], r2 = c.linear ? 0.0f : c.r2[h];
-  float m = c.sink[h], l = 1.0f;
+  const float r1 = c.bias == 2 ? 0.0f : c.r1[h], r2 = c.bias ? 0.0f : c.r2[h];
+  float m = c.sink ? c.sink[h] : -INFINITY, l = c.sink ? 1.0f : 0.0f;
   float acc[HY_ATT_MAXD];
 #pragma unroll
   for (int i = 0; i < HY_ATT_MAXD; ++i) acc[i] = 0.0f;
@@ -294,7 +296,7 @@ __global__ void __launch_bounds__(128) biased_attn_kernel(Batch b, const AT* __r
       for (int d = 0; d < c.dim; ++d) dot = fmaf(qs[d], to_f(kr[d]), dot);
       s = dot * c.scale;
       if (c.cap > 0.0f) s = c.cap * tanhf(s / c.cap);
-      s -= r1 * (c.linear ? (float)(pos - j) : log1pf(r2 * (float)(pos - j)));
+      if (c.bias != 2) s -= r1 * (c.bias == 1 ? (float)(pos - j) : log1pf(r2 * (float)(pos - j)));
     }
     const float mn = fmaxf(m, warp_max(s));
     const float corr = expf(m - mn);
@@ -315,7 +317,7 @@ __global__ void __launch_bounds__(128) biased_attn_kernel(Batch b, const AT* __r
       }
     }
   }
-  const float inv = 1.0f / l;
+  const float inv = c.out_factor(t, h) / l;
 #pragma unroll
   for (int i = 0; i < HY_ATT_MAXD; ++i) {
     const int d = lane + 32 * i;
@@ -371,7 +373,8 @@ __global__ void __launch_bounds__(128) biased_mma_kernel(Batch b, const AttnUnit
   const bool v_lo = r_lo < rows_total, v_hi = r_hi < rows_total;
   const int p_lo = v_lo ? pos0 + r_lo / R : -1, p_hi = v_hi ? pos0 + r_hi / R : -1;
   const int h_lo = u.kv_head * R + r_lo % R, h_hi = u.kv_head * R + r_hi % R;
-  const float r1_lo = c.r1[h_lo], r2_lo = c.linear ? 0.0f : c.r2[h_lo], r1_hi = c.r1[h_hi], r2_hi = c.linear ? 0.0f : c.r2[h_hi];
+  const float r1_lo = c.bias == 2 ? 0.0f : c.r1[h_lo], r1_hi = c.bias == 2 ? 0.0f : c.r1[h_hi];
+  const float r2_lo = c.bias ? 0.0f : c.r2[h_lo], r2_hi = c.bias ? 0.0f : c.r2[h_hi];
   const int f_lo = c.first(max(p_lo, 0)), f_hi = c.first(max(p_hi, 0));                           // first visible position of each row
   const bool warp_live = (u.row0 + warp * 16) < rows_total;
   const float inv_cap = c.cap > 0.0f ? 1.0f / c.cap : 0.0f;
@@ -446,10 +449,10 @@ __global__ void __launch_bounds__(128) biased_mma_kernel(Batch b, const AttnUnit
           a = c.cap * (1.0f - __fdividef(2.0f, __expf(2.0f * a * inv_cap) + 1.0f));
           d = c.cap * (1.0f - __fdividef(2.0f, __expf(2.0f * d * inv_cap) + 1.0f));
         }
-        if (c.linear) {
+        if (c.bias == 1) {
           a = fmaf(-r1_lo, (float)(p_lo - j), a);
           d = fmaf(-r1_hi, (float)(p_hi - j), d);
-        } else {
+        } else if (c.bias == 0) {
           a -= r1_lo * __logf(fmaf(r2_lo, (float)(p_lo - j), 1.0f));
           d -= r1_hi * __logf(fmaf(r2_hi, (float)(p_hi - j), 1.0f));
         }
@@ -534,10 +537,10 @@ __global__ void __launch_bounds__(128) biased_mma_kernel(Batch b, const AttnUnit
       continue;
     }
     // the sink: one more term in the denominator
-    const float m = hh ? m_hi : m_lo, sk = c.sink[h];
+    const float m = hh ? m_hi : m_lo, sk = c.sink ? c.sink[h] : -INFINITY;
     const float top = fmaxf(m, sk);
     const float f = expf(m - top);
-    const float inv = f / ((hh ? l_hi : l_lo) * f + expf(sk - top));
+    const float inv = f * c.out_factor(t, h) / ((hh ? l_hi : l_lo) * f + expf(sk - top));
     bf16* po = out + (size_t)t * ldo + h * c.vdim;
 #pragma unroll
     for (int i = 0; i < DP / 8; ++i) {
@@ -551,16 +554,17 @@ __global__ void __launch_bounds__(128) biased_mma_kernel(Batch b, const AttnUnit
 // Merge the key splits of one (token, head) with the sink: one block per (token, head).  A split without keys holds a
 // maximum of -inf and a denominator of zero.  part_o rows are pstride wide.
 template <typename OT>
-__global__ void biased_combine_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml, const float* __restrict__ sink,
-                                      int H, int vdim, int pstride, int n_splits, OT* __restrict__ out, int ldo) {
+__global__ void biased_combine_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml, BiasedCfg c,
+                                      int pstride, int n_splits, OT* __restrict__ out, int ldo) {
+  const int H = c.H, vdim = c.vdim;
   const int t = blockIdx.x / H, h = blockIdx.x % H;
   const size_t slot0 = ((size_t)t * H + h) * n_splits;
-  const float sk = sink[h];
+  const float sk = c.sink ? c.sink[h] : -INFINITY;
   float M = sk;
   for (int s = 0; s < n_splits; ++s) M = fmaxf(M, part_ml[(slot0 + s) * 2]);
   float L = expf(sk - M);
   for (int s = 0; s < n_splits; ++s) L += part_ml[(slot0 + s) * 2 + 1] * expf(part_ml[(slot0 + s) * 2] - M);
-  const float inv = 1.0f / L;
+  const float inv = c.out_factor(t, h) / L;
   for (int d = threadIdx.x; d < vdim; d += blockDim.x) {
     float acc = 0.0f;
     for (int s = 0; s < n_splits; ++s) acc += part_o[(slot0 + s) * pstride + d] * expf(part_ml[(slot0 + s) * 2] - M);

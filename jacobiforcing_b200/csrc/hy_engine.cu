@@ -23,6 +23,7 @@
 #include "hy_experts.cuh"
 #include "hy_window.cuh"
 #include "hy_biased.cuh"
+#include "hy_delta.cuh"
 #include "hy_gla.cuh"
 
 namespace hy {
@@ -90,6 +91,10 @@ struct LayerW {
   // in w_in, and as tiles [mixer columns padded to 32 | 16 gate / 16 up alternating | fp32 columns]; the fp32 columns are the
   // latent's down-projection or the decay projection's first step, then the router's outputs
   int n_mix = 0, n_f32 = 0, c_router = 0, t_pair = 0; float* x_corr = nullptr;
+  // norm - sublayer - norm blocks with plain RMS weights (norm1 above): the other three norms; retention's decays; the cosine / sine
+  // table of the layer's rotation (index into hy_engine.rot_tables)
+  void* norm1b = nullptr; void* norm2 = nullptr; void* norm2b = nullptr;
+  float* decay = nullptr; int rot_table = -1;
 };
 
 // One layer run of a step: the layer of the checkpoint and whether a pass of a repeated span begins with it.
@@ -150,6 +155,10 @@ struct hy_engine {
   // tensor-core attention: work units of the step (per head layout), partial results per (row, key split)
   AttnUnit* units_d = nullptr; AttnUnit* units_h = nullptr; size_t units_cap = 0, units_used = 0;
   std::vector<UnitList> unit_lists;
+  // cosines and sines of the step's positions, one table per distinct rotation: the layer configuration that names it, the table,
+  // its column count; rot_tables_d is what the kernel reads
+  struct RotEntry { hy_layer_cfg c; RotTable t; };
+  std::vector<RotEntry> rot_tables; RotTable* rot_tables_d = nullptr;
   float* part_o = nullptr; float* part_ml = nullptr; size_t part_rows = 0, part_dim = 0;
   const int32_t* step_start = nullptr; const int32_t* step_pos0 = nullptr;     // host views of the running step
   size_t esz() const { return m.dtype == HY_DTYPE_F32 ? 4 : 2; }
@@ -212,6 +221,7 @@ extern "C" int hy_create(const hy_model_cfg* model, const hy_layer_cfg* layers, 
   if (model->loop_times > 0 && (model->loop_start < 0 || model->loop_start >= model->loop_stop || model->loop_stop > model->n_layers))
     return bad("repeated layers: 0 <= start < stop <= layers");
   const bool rms_parallel = model->block_kind == HY_BLOCK_PARALLEL && model->norm_kind == HY_NORM_RMS;
+  const bool rms_sandwich = model->block_kind == HY_BLOCK_SANDWICH && model->norm_kind == HY_NORM_RMS;
   if (model->loop_times > 0 && !rms_parallel) return bad("repeated layers need one-norm-per-layer blocks with plain RMS weights");
   if (rt->page_size <= 0 || rt->page_size % 16) return bad("page_size must be a positive multiple of 16");
   for (auto& c : h->lc) {
@@ -235,8 +245,10 @@ extern "C" int hy_create(const hy_model_cfg* model, const hy_layer_cfg* layers, 
       if (c.l_heads <= 0 || c.l_dim <= 0 || c.l_vdim <= 0 || c.l_kv_rank <= 0 || c.l_q_rank < 0 || c.l_rot_dim < 0) return bad("latent attention sizes must be positive");
       if (c.l_kv_rank + c.l_rot_dim > 32 * HY_ATT_MAXD) return bad("latent rank + rotated size above 640");
       if (c.r_dims < 0 || c.r_dims % 2 || c.r_dims > c.l_rot_dim) return bad("rotated dimensions must be even and at most rot_dim");
-      if (rms_parallel != (c.l_q_rank == 0)) return bad("full-rank queries belong to one-norm-per-layer blocks, a query latent to the others");
-      if (rms_parallel && (c.l_kv_from >= 0 || !c.l_no_sink)) return bad("latent attention of this block layout has a latent of its own and no sink");
+      if ((rms_parallel || rms_sandwich) != (c.l_q_rank == 0)) return bad("full-rank queries belong to blocks with plain RMS weights, a query latent to the others");
+      if ((rms_parallel || rms_sandwich) && (c.l_kv_from >= 0 || !c.l_no_sink)) return bad("latent attention of this block layout has a latent of its own and no sink");
+      if (c.l_window < 0) return bad("the window must not be negative");
+      if (c.l_gate && !rms_sandwich) return bad("a gated latent attention belongs to norm - sublayer - norm blocks with plain RMS weights");
       const int idx = (int)(&c - h->lc.data());
       if (c.l_kv_from >= 0) {
         if (c.l_kv_from >= idx) return bad("a borrowed latent must come from an earlier layer");
@@ -270,11 +282,24 @@ extern "C" int hy_create(const hy_model_cfg* model, const hy_layer_cfg* layers, 
       if (c.g_heads <= 0 || c.g_dim <= 0 || c.g_vdim <= 0 || c.g_low <= 0) return bad("gated linear attention sizes must be positive");
       if (c.g_dim > 1024) return bad("gated linear attention: key size above 1024");
       if (!(c.g_tau > 0.0f)) return bad("gated linear attention: tau must be positive");
+    } else if (c.mixer == HY_MIX_RETENTION) {
+      if (c.g_heads <= 0 || c.g_dim <= 0 || c.g_vdim <= 0 || c.g_dim > 1024) return bad("retention: sizes must be positive, the key size at most 1024");
+      if (c.r_dims < 0 || c.r_dims % 2 || c.r_dims > c.g_dim) return bad("rotated dimensions must be even and at most dim");
+    } else if (c.mixer == HY_MIX_ATTN_DELTA) {
+      if (c.b_heads <= 0 || c.b_kv_heads <= 0 || c.b_heads % c.b_kv_heads) return bad("attention heads must be a multiple of kv_heads");
+      if (c.b_dim <= 0 || c.b_dim > 32 * HY_ATT_MAXD || c.b_vdim != c.b_dim) return bad("attention whose values are its keys: vdim == dim, in 1..640");
+      if (c.b_bias != HY_BIAS_NONE || c.b_window || c.b_keep_first || c.b_chunk || c.b_softcap > 0.0f) return bad("attention of this mixer is causal over all keys, without bias and cap");
+      if (c.r_dims < 0 || c.r_dims % 2 || c.r_dims > c.b_dim) return bad("rotated dimensions must be even and at most dim");
+      if (c.d_heads <= 0 || c.d_kv_heads <= 0 || c.d_heads % c.d_kv_heads) return bad("delta heads must be a multiple of kv_heads");
+      if (c.d_dim <= 0 || c.d_vdim <= 0 || c.d_dim > 1024) return bad("delta rule: sizes must be positive, the key size at most 1024");
+      if (c.d_conv > HY_MAX_TAPS || c.d_conv < 1) return bad("conv taps must lie in 1..16");
     } else {
       return bad("unknown mixer kind");
     }
     const bool any_block = rms_parallel && (c.mixer == HY_MIX_LATENT || c.mixer == HY_MIX_BIASED || c.mixer == HY_MIX_GLA);
-    const int mixer_block = any_block ? HY_BLOCK_PARALLEL : (c.mixer == HY_MIX_SSD || c.mixer == HY_MIX_LATENT || c.mixer == HY_MIX_GLR) ? HY_BLOCK_SANDWICH
+    const bool rms_mixer = c.mixer == HY_MIX_RETENTION || c.mixer == HY_MIX_ATTN_DELTA || c.mixer == HY_MIX_LATENT;
+    if (rms_sandwich ? !rms_mixer : c.mixer == HY_MIX_RETENTION || c.mixer == HY_MIX_ATTN_DELTA) return bad("this mixer does not belong to the model's block layout");
+    const int mixer_block = rms_sandwich ? HY_BLOCK_SANDWICH : any_block ? HY_BLOCK_PARALLEL : (c.mixer == HY_MIX_SSD || c.mixer == HY_MIX_LATENT || c.mixer == HY_MIX_GLR) ? HY_BLOCK_SANDWICH
                             : (c.mixer == HY_MIX_WINDOW || c.mixer == HY_MIX_MLSTM) ? HY_BLOCK_POSTNORM
                             : c.mixer == HY_MIX_BIASED ? HY_BLOCK_PRENORM : HY_BLOCK_PARALLEL;
     if (mixer_block != model->block_kind || rms_parallel != any_block) return bad("this mixer does not belong to the model's block layout");
@@ -283,17 +308,20 @@ extern "C" int hy_create(const hy_model_cfg* model, const hy_layer_cfg* layers, 
                          (c.ff_kind == HY_FF_GATED && (rms_parallel || model->block_kind == HY_BLOCK_POSTNORM || model->block_kind == HY_BLOCK_PRENORM));
     if (!ff_fits) return bad("this feed-forward does not belong to the model's block layout");
     if (c.ff_kind == HY_FF_ROUTED) {
-      if (c.x_experts <= 0 || c.x_experts > 4096 || c.x_groups <= 0 || c.x_experts % c.x_groups) return bad("experts must split into equal groups");
+      const int outputs = c.x_experts + (c.x_route == HY_ROUTE_CORRECTED_SOFTMAX ? c.x_identity : 0);
+      if (c.x_experts <= 0 || c.x_experts > 4096 || c.x_groups <= 0 || outputs % c.x_groups) return bad("router outputs must split into equal groups");
       if (c.x_keep < 1 || c.x_keep > c.x_groups) return bad("kept groups outside 1..groups");
       if (c.x_identity < 0 || c.x_identity > 1024 || (c.x_identity > 0 && c.x_route != HY_ROUTE_CORRECTED_SOFTMAX))
         return bad("identity experts go with corrected softmax scores");
-      if (c.x_top < 1 || c.x_top > (c.x_route == HY_ROUTE_CORRECTED_SOFTMAX ? c.x_experts + c.x_identity : c.x_keep * (c.x_experts / c.x_groups))) return bad("more experts per token than the kept groups hold");
+      if (c.x_top < 1 || c.x_top > c.x_keep * (outputs / c.x_groups)) return bad("more experts per token than the kept groups hold");
       if (c.ff <= 0) return bad("expert size must be positive");
       if (c.x_route < HY_ROUTE_SIGMOID_GROUPS || c.x_route > HY_ROUTE_CORRECTED_SOFTMAX) return bad("unknown router kind");
       if (rms_parallel && (c.x_plain || c.x_shared_ff || c.x_route != HY_ROUTE_CORRECTED_SOFTMAX))
         return bad("one-norm-per-layer blocks serve gated experts with corrected softmax scores only");
       if (c.x_act < 0 || c.x_act > 3 || (c.x_act == HY_ACT_CLAMPED && c.x_plain) || c.x_shared_ff < 0) return bad("unknown expert activation or negative shared size");
-      if (model->block_kind == HY_BLOCK_SANDWICH && (c.x_plain || c.x_shared_ff || c.x_route || c.x_act))
+      if (rms_sandwich && (c.x_plain || c.x_shared_ff || c.x_route != HY_ROUTE_CORRECTED_SOFTMAX))
+        return bad("norm - sublayer - norm blocks with plain RMS weights serve gated experts with corrected softmax scores only");
+      if (!rms_sandwich && model->block_kind == HY_BLOCK_SANDWICH && (c.x_plain || c.x_shared_ff || c.x_route || c.x_act))
         return bad("norm - sublayer - norm blocks serve gated silu experts with sigmoid scores only");
       if (model->block_kind == HY_BLOCK_POSTNORM && !c.x_plain) return bad("output-normed blocks serve experts without a gate only");
       if (model->block_kind == HY_BLOCK_PRENORM && (c.x_plain || c.x_shared_ff || c.x_route != HY_ROUTE_TOP_SOFTMAX))
@@ -307,7 +335,7 @@ extern "C" int hy_create(const hy_model_cfg* model, const hy_layer_cfg* layers, 
   }
   const int want_norm = model->block_kind == HY_BLOCK_SANDWICH ? HY_NORM_TANH
                         : (model->block_kind == HY_BLOCK_POSTNORM || model->block_kind == HY_BLOCK_PRENORM) ? HY_NORM_RMS : HY_NORM_RMS_OFFSET;
-  if (model->norm_kind != want_norm && !rms_parallel) return bad("block layout and norm kind do not go together");
+  if (model->norm_kind != want_norm && !rms_parallel && !rms_sandwich) return bad("block layout and norm kind do not go together");
   if (cudaSetDevice(rt->device) != cudaSuccess) return bad("cudaSetDevice failed");
   cudaStreamCreate(&h->stream);
   cudaEventCreate(&h->ev0);
@@ -475,8 +503,12 @@ bool tanh_norm_load(Builder& B, const std::string& name, int W, TanhNorm* n) {
 int load_gated_experts(hy_engine* h, Builder& B, LayerW& L, const hy_layer_cfg& c, const std::string& p, Maxima& mx) {
   const int W = h->m.width;
   const int E = c.x_experts, ff = c.ff;
-  if (c.x_route != HY_ROUTE_CORRECTED_SOFTMAX) {              // the corrected scores' router sits in the merged input projection
-    if (auto t = B.get(p + "mlp.router", E, W)) { L.w_router = B.up(t->v); L.w_router_t = B.up_tiled(t->v, E, W); }
+  const bool corrected = c.x_route == HY_ROUTE_CORRECTED_SOFTMAX;
+  if (!corrected || h->m.block_kind != HY_BLOCK_PARALLEL) {   // one-norm-per-layer blocks: the router sits in the merged input projection
+    const int outputs = E + (corrected ? c.x_identity : 0);
+    if (auto t = B.get(p + "mlp.router", outputs, W)) { L.w_router = B.up(t->v); L.w_router_t = B.up_tiled(t->v, outputs, W); }
+    if (corrected) { if (auto t = B.get(p + "mlp.correction", outputs, -1)) L.x_corr = B.up_f32(t->v); }
+    mx.f1 = std::max(mx.f1, outputs);
   }
   std::vector<float> gu, dn;
   gu.reserve((size_t)E * 2 * ff * W);
@@ -1010,6 +1042,128 @@ int finalize_parallel_layer(hy_engine* h, Builder& B, size_t i, Maxima& mx) {
   return alloc_parallel_memory(h, L, c);
 }
 
+// Index of the cosine / sine table of a layer's rotation; layers with the same rotation share one.
+int rotation_table_of(hy_engine* h, Builder& B, const hy_layer_cfg& c, LayerW& L) {
+  for (size_t i = 0; i < h->rot_tables.size(); ++i) {
+    const hy_layer_cfg& o = h->rot_tables[i].c;
+    if (o.r_dims == c.r_dims && o.r_base == c.r_base && o.r_factor == c.r_factor && o.r_original == c.r_original && o.r_fast == c.r_fast &&
+        o.r_slow == c.r_slow) { L.rot_table = (int)i; return HY_OK; }
+  }
+  std::vector<double> f;
+  RotTable t{};
+  rotation_table(c, f, &t.mag);
+  t.pairs = (int)f.size();
+  t.ld = (2 * t.pairs + 3) & ~3;
+  void* d = nullptr;
+  if (dev_alloc(h, &d, f.size() * 8, &h->bytes_w)) return HY_ERR_CUDA;
+  cudaMemcpy(d, f.data(), f.size() * 8, cudaMemcpyHostToDevice);
+  t.freq = (const double*)d;
+  if (dev_alloc(h, (void**)&t.out, (size_t)h->rt.max_step_tokens * t.ld * 4, &h->bytes_ws)) return HY_ERR_CUDA;
+  L.rot_table = (int)h->rot_tables.size();
+  h->rot_tables.push_back({c, t});
+  return B.rc;
+}
+
+// One layer of a norm - sublayer - norm model with plain RMS weights: four norms, the mixer's merged input projection (operand
+// columns, then the columns that leave as fp32), its small tensors, the merged output projection, cache and state, the experts.
+int finalize_rms_sandwich_layer(hy_engine* h, Builder& B, size_t i, Maxima& mx) {
+  const hy_layer_cfg& c = h->lc[i];
+  const hy_runtime_cfg& rt = h->rt;
+  LayerW& L = h->lw[i];
+  const int W = h->m.width;
+  const size_t tokens = (size_t)rt.num_pages * rt.page_size;
+  const std::string p = "l" + std::to_string(i) + ".", d = p + "mix.";
+  if (auto t = B.get(p + "norm1", W, -1)) L.norm1 = B.up(t->v);
+  if (auto t = B.get(p + "norm1b", W, -1)) L.norm1b = B.up(t->v);
+  std::vector<float> win;
+  std::vector<const HostTensor*> outs;                        // output projections, merged along k
+  if (c.mixer == HY_MIX_RETENTION) {
+    const int H = c.g_heads, nq = H * c.g_dim, nv = H * c.g_vdim;
+    L.c_q = 0; L.c_k = nq; L.c_v = 2 * nq; L.c_g = 2 * nq + nv;
+    L.n_mix = 2 * nq + 2 * nv;
+    stack_rows(win, B.get(d + "q", nq, W));
+    stack_rows(win, B.get(d + "k", nq, W));
+    stack_rows(win, B.get(d + "v", nv, W));
+    stack_rows(win, B.get(d + "g", nv, W));
+    if (auto t = B.get(d + "decay", H, -1)) L.decay = B.up_f32(t->v);
+    outs.push_back(B.get(d + "o", W, nv));
+    if (int rc = rotation_table_of(h, B, c, L)) return rc;
+    mx.f2 = std::max(mx.f2, nv);
+    if (dev_alloc(h, (void**)&L.rec_state, (size_t)rt.num_slots * H * c.g_dim * c.g_vdim * 4, &h->bytes_state)) return HY_ERR_CUDA;
+  } else if (c.mixer == HY_MIX_ATTN_DELTA) {
+    const std::string a = d + "left.", r = d + "right.";
+    const int H = c.b_heads, G = c.b_kv_heads, nq = H * c.b_dim, nk = G * c.b_dim;
+    const int Hd = c.d_heads, dk = c.d_kv_heads * c.d_dim, dv = Hd * c.d_vdim, C = 2 * dk + dv;
+    L.c_q = 0; L.c_k = nq; L.c_x = nq + nk; L.c_g = L.c_x + C;
+    L.n_mix = L.c_g + dv;
+    stack_rows(win, B.get(a + "q", nq, W));
+    stack_rows(win, B.get(a + "k", nk, W));
+    stack_rows(win, B.get(r + "q", dk, W));
+    stack_rows(win, B.get(r + "k", dk, W));
+    stack_rows(win, B.get(r + "v", dv, W));
+    stack_rows(win, B.get(r + "g", dv, W));
+    stack_rows(win, B.get(a + "g", H, W));                    // fp32 columns: head gates, step sizes, decays
+    stack_rows(win, B.get(r + "b", Hd, W));
+    stack_rows(win, B.get(r + "a", Hd, W));
+    L.n_f32 = H + 2 * Hd;
+    std::vector<float> cw;
+    stack_rows(cw, B.get(r + "q.conv", dk, c.d_conv));
+    stack_rows(cw, B.get(r + "k.conv", dk, c.d_conv));
+    stack_rows(cw, B.get(r + "v.conv", dv, c.d_conv));
+    L.conv_qkv = B.up(cw);
+    if (auto t = B.get(r + "A_log", Hd, -1)) L.A_log = B.up_f32(t->v);
+    if (auto t = B.get(r + "dt_bias", Hd, -1)) L.dt_bias = B.up_f32(t->v);
+    if (auto t = B.get(r + "norm", c.d_vdim, -1)) L.g_norm = B.up_f32(t->v);
+    outs.push_back(B.get(a + "o", W, nq));
+    outs.push_back(B.get(r + "o", W, dv));
+    if (int rc = rotation_table_of(h, B, c, L)) return rc;
+    mx.cv = std::max(mx.cv, C);
+    mx.f2 = std::max(mx.f2, dv);
+    if (dev_alloc(h, &L.cache, tokens * nk * h->esz(), &h->bytes_cache)) return HY_ERR_CUDA;
+    if (dev_alloc(h, &L.cache_v, tokens * nk * h->esz(), &h->bytes_cache)) return HY_ERR_CUDA;
+    if (dev_alloc(h, (void**)&L.conv_state, (size_t)rt.num_slots * (c.d_conv - 1) * C * 4, &h->bytes_state)) return HY_ERR_CUDA;
+    if (dev_alloc(h, (void**)&L.rec_state, (size_t)rt.num_slots * dv * c.d_dim * 4, &h->bytes_state)) return HY_ERR_CUDA;
+  } else {
+    const int H = c.l_heads, R = c.l_kv_rank, Dk = R + c.l_rot_dim, nq = H * (c.l_dim + c.l_rot_dim), nv = H * c.l_vdim;
+    L.c_g = nq;
+    L.n_mix = nq + (c.l_gate ? nv : 0);
+    stack_rows(win, B.get(d + "q", nq, W));
+    if (c.l_gate) stack_rows(win, B.get(d + "g", nv, W));
+    stack_rows(win, B.get(d + "dkv", Dk, W));
+    L.n_f32 = Dk;
+    if (auto t = B.get(d + "dkv.norm", R, -1)) L.l_kn = B.up_f32(t->v);
+    if (int rc = load_latent_up(h, B, L, c, d)) return rc;
+    outs.push_back(B.get(d + "o", W, nv));
+    mx.cv = std::max(mx.cv, H * Dk);
+    mx.f2 = std::max(mx.f2, H * R);
+    if (dev_alloc(h, &L.cache, tokens * Dk * h->esz(), &h->bytes_cache)) return HY_ERR_CUDA;
+  }
+  if (B.rc != HY_OK) return B.rc;
+  L.n_in = L.n_mix + L.n_f32;
+  L.w_in = B.up(win);
+  L.w_in_t = B.up_tiled(win, L.n_in, W);
+  L.k_out = 0;
+  for (auto t : outs) L.k_out += (int)t->cols();
+  std::vector<float> wout((size_t)W * L.k_out);
+  int off = 0;
+  for (auto t : outs) {
+    const int kc = (int)t->cols();
+    for (int r = 0; r < W; ++r) memcpy(&wout[(size_t)r * L.k_out + off], &t->v[(size_t)r * kc], (size_t)kc * 4);
+    off += kc;
+  }
+  L.o_mix = 0; L.o_scan = outs[0]->cols();
+  L.w_out = B.up(wout);
+  L.w_out_t = B.up_tiled(wout, W, L.k_out);
+  mx.in = std::max(mx.in, L.n_mix);
+  mx.out = std::max(mx.out, L.k_out);
+  mx.f1 = std::max(mx.f1, L.n_f32);
+  mx.f2 = std::max(mx.f2, W);
+  if (c.ff_kind == HY_FF_NONE) return B.rc;
+  if (auto t = B.get(p + "norm2", W, -1)) L.norm2 = B.up(t->v);
+  if (auto t = B.get(p + "norm2b", W, -1)) L.norm2b = B.up(t->v);
+  return load_gated_experts(h, B, L, c, p, mx);
+}
+
 // rows of several [n_i, k] matrices stacked
 void stack_rows(std::vector<float>& dst, const HostTensor* t) { if (t) dst.insert(dst.end(), t->v.begin(), t->v.end()); }
 
@@ -1053,7 +1207,8 @@ extern "C" int hy_finalize(hy_handle h) {
     const hy_layer_cfg& c = h->lc[i];
     LayerW& L = h->lw[i];
     if (h->m.block_kind != HY_BLOCK_PARALLEL || h->m.norm_kind == HY_NORM_RMS) {
-      const int rc = h->m.block_kind == HY_BLOCK_PARALLEL ? finalize_parallel_layer(h, B, i, mx) : h->m.block_kind == HY_BLOCK_SANDWICH ? finalize_sandwich_layer(h, B, i, mx)
+      const int rc = h->m.block_kind == HY_BLOCK_PARALLEL ? finalize_parallel_layer(h, B, i, mx)
+                     : h->m.block_kind == HY_BLOCK_SANDWICH ? (h->m.norm_kind == HY_NORM_RMS ? finalize_rms_sandwich_layer(h, B, i, mx) : finalize_sandwich_layer(h, B, i, mx))
                      : h->m.block_kind == HY_BLOCK_POSTNORM ? finalize_postnorm_layer(h, B, i, mx) : finalize_prenorm_layer(h, B, i, mx);
       if (rc != HY_OK) return rc;
       continue;
@@ -1186,12 +1341,12 @@ extern "C" int hy_finalize(hy_handle h) {
     std::set<std::vector<int>> layouts;                      // attention layouts whose unit lists one step may hold
     for (auto& c : h->lc) {
       if (c.mixer == HY_MIX_ATTN_SCAN) layouts.insert({1, c.a_heads, c.a_kv_heads});
-      if (c.mixer == HY_MIX_LATENT) layouts.insert({1, c.l_heads, 1});
+      if (c.mixer == HY_MIX_LATENT) layouts.insert({1, c.l_heads, 1, c.l_window});
       if (c.mixer == HY_MIX_WINDOW) layouts.insert({2, c.w_heads, c.w_kv_heads});
-      if (c.mixer == HY_MIX_BIASED) layouts.insert({3, c.b_heads, c.b_kv_heads, c.b_window, c.b_chunk});
+      if (c.mixer == HY_MIX_BIASED || c.mixer == HY_MIX_ATTN_DELTA) layouts.insert({3, c.b_heads, c.b_kv_heads, c.b_window, c.b_chunk});
       if (c.mixer == HY_MIX_ATTN_SCAN) { maxH = std::max(maxH, c.a_heads); maxG = std::max(maxG, c.a_kv_heads); maxD = std::max(maxD, c.a_dim); }
       if (c.mixer == HY_MIX_WINDOW) { maxH = std::max(maxH, c.w_heads); maxG = std::max(maxG, c.w_kv_heads); maxD = std::max(maxD, 8); }
-      if (c.mixer == HY_MIX_BIASED) {                       // partial rows of the key splits are one tile row wide
+      if (c.mixer == HY_MIX_BIASED || c.mixer == HY_MIX_ATTN_DELTA) {   // partial rows of the key splits are one tile row wide
         maxH = std::max(maxH, c.b_heads); maxG = std::max(maxG, c.b_kv_heads);
         maxD = std::max(maxD, (c.b_dim <= 64 && c.b_vdim <= 64) ? 64 : 128);
       }
@@ -1230,6 +1385,12 @@ extern "C" int hy_finalize(hy_handle h) {
       HY_CUDA(cudaMemset(h->x_counts, 0, (size_t)maxE * 4));
       HY_CUDA(cudaMemset(h->x_meta, 0, 16));
     }
+  }
+  if (!h->rot_tables.empty()) {
+    std::vector<RotTable> t;
+    for (auto& r : h->rot_tables) t.push_back(r.t);
+    if (dev_alloc(h, (void**)&h->rot_tables_d, t.size() * sizeof(RotTable), &h->bytes_ws)) return HY_ERR_CUDA;
+    HY_CUDA(cudaMemcpy(h->rot_tables_d, t.data(), t.size() * sizeof(RotTable), cudaMemcpyHostToDevice));
   }
   if (dev_alloc(h, (void**)&h->err_d, 4, &h->bytes_ws)) return HY_ERR_CUDA;
   HY_CUDA(cudaMemset(h->err_d, 0, 4));
@@ -1332,27 +1493,38 @@ struct UnitWriter {
 
 // Work units of the tensor-core attention for this step and this head layout; NULL when the layout does not fit the kernel
 // (the SIMT kernel serves it then).  The pointer holds until the next list is made.
-const UnitList* attn_units(hy_engine* h, int E, int T, int H, int G, bool any_ratio = false) {
+// With a sliding window a tile has units only for the key splits from the one its first row's window begins in (see first_split);
+// the splits are cut for the keys a tile sees, so a tile meets at most one more of them than there are.
+const UnitList* attn_units(hy_engine* h, int E, int T, int H, int G, bool any_ratio = false, int window = 0) {
   const int R = H / G;
   if (!any_ratio && (R > 64 || 64 % R)) return nullptr;
-  if (const UnitList* u = find_units(h, 1, H, G, 0, 0)) return u;
+  if (const UnitList* u = find_units(h, 1, H, G, window, 0)) return u;
   int maxctx = 1;
   for (int e = 0; e < E; ++e) maxctx = std::max(maxctx, h->step_pos0[e] + h->step_start[e + 1] - h->step_start[e]);
   const int ns_cap = (int)std::max<size_t>(1, h->part_rows / ((size_t)T * H));
   int ns = std::min(std::min((maxctx + 255) / 256, ns_cap), 256);
-  const int split = ((maxctx + ns - 1) / ns + 63) / 64 * 64;
+  int split = ((maxctx + ns - 1) / ns + 63) / 64 * 64;
   ns = (maxctx + split - 1) / split;
+  const int seen = window > 0 ? window + 63 / R : maxctx;     // most keys a tile of 64 rows sees
+  if (seen < maxctx && ns_cap >= 2) {
+    const int n = std::min(std::min((seen + 255) / 256, ns_cap - 1), 255);
+    split = ((seen + n - 1) / n + 63) / 64 * 64;
+    ns = std::min((seen + split - 1) / split + 1, (maxctx + split - 1) / split);
+  } else if (seen < maxctx) {
+    split = (maxctx + 63) / 64 * 64;
+    ns = 1;
+  }
   UnitWriter w(h);
   for (int e = 0; e < E; ++e) {
     const int cnt = h->step_start[e + 1] - h->step_start[e], pos0 = h->step_pos0[e], rows = cnt * R;
     for (int g = 0; g < G; ++g)
       for (int row0 = (rows - 1) / 64 * 64; row0 >= 0; row0 -= 64) {          // late rows see the most keys: start them first
-        const int last_pos = pos0 + std::min(row0 + 63, rows - 1) / R;
-        for (int sp = 0; sp * split <= last_pos; ++sp)
-          if (!w.add(AttnUnit{e, g, row0, sp})) return nullptr;
+        const int last_pos = pos0 + std::min(row0 + 63, rows - 1) / R, sp0 = first_split(pos0 + row0 / R, window, split);
+        for (int sp = 0; (sp0 + sp) * split <= last_pos; ++sp)
+          if (sp >= ns || !w.add(AttnUnit{e, g, row0, sp})) return nullptr;
       }
   }
-  return w.commit(1, H, G, 0, 0, split, ns);
+  return w.commit(1, H, G, window, 0, split, ns);
 }
 
 // Work units of the tensor-core window attention: (entry, key head, tile of 64 rows), late tiles first (they see the most).
@@ -1438,22 +1610,22 @@ void latent_mixer(hy_engine* h, const Batch& b, const LayerW& L, const hy_layer_
     const UnitList* u = nullptr;
     (void)u;
     if constexpr (std::is_same<AT, bf16>::value) {
-      if ((Dk == 32 || Dk == 64 || Dk == 128) && h->part_o && (u = attn_units(h, E, T, H, 1))) {
+      if ((Dk == 32 || Dk == 64 || Dk == 128) && h->part_o && (u = attn_units(h, E, T, H, 1, false, c.l_window))) {
         tc = true;
-#define HY_ATTN_ARGS b, u->d, cv, h->ld_cv, (const bf16*)L.cache, H, 1, c.l_scale, 0.0f, 1, u->split, u->ns, R, \
+#define HY_ATTN_ARGS b, u->d, cv, h->ld_cv, (const bf16*)L.cache, H, 1, c.l_scale, 0.0f, 1, c.l_window, u->split, u->ns, R, \
         h->part_o, h->part_ml
         if (Dk == 32) attn_mma_kernel<32><<<u->n, 128, 0, s>>>(HY_ATTN_ARGS);
         else if (Dk == 64) attn_mma_kernel<64><<<u->n, 128, 0, s>>>(HY_ATTN_ARGS);
         else attn_mma_kernel<128><<<u->n, 128, 0, s>>>(HY_ATTN_ARGS);
 #undef HY_ATTN_ARGS
-        attn_combine_kernel<WT, float><<<T * H, 64, 0, s>>>(b, h->part_o, h->part_ml, (const WT*)L.sink, nullptr, 0, H, Dk, R,
-                                                            u->split, u->ns, 1.0f, h->f2, h->ld_f2);
+        attn_combine_kernel<WT, float><<<T * H, 64, 0, s>>>(b, h->part_o, h->part_ml, (const WT*)L.sink, nullptr, 0, H, 1, Dk, R,
+                                                            c.l_window, u->split, u->ns, 1.0f, h->f2, h->ld_f2);
         h->launches += 2;
       }
     }
     if constexpr (std::is_same<AT, bf16>::value) {
       // wide cache rows (or a head count the narrow kernel does not tile): eight warps per tile, values split by warp
-      if (!tc && Dk % 8 == 0 && R <= 512 && h->part_o && (u = attn_units(h, E, T, H, 1, true))) {
+      if (!tc && Dk % 8 == 0 && R <= 512 && h->part_o && (u = attn_units(h, E, T, H, 1, true, c.l_window))) {
         tc = true;
         const int nt = R <= 128 ? 2 : R <= 256 ? 4 : 8, pstride = nt * 64;
         const size_t smem = attn_wide_smem(Dk);
@@ -1464,32 +1636,33 @@ void latent_mixer(hy_engine* h, const Batch& b, const LayerW& L, const hy_layer_
           cudaFuncSetAttribute(attn_wide_kernel<8>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)attn_wide_smem(640));
           wide_attr = true;
         }
-#define HY_WIDE_ARGS b, u->d, cv, h->ld_cv, (const bf16*)L.cache, H, Dk, R, c.l_scale, u->split, u->ns, pstride, \
+#define HY_WIDE_ARGS b, u->d, cv, h->ld_cv, (const bf16*)L.cache, H, Dk, R, c.l_scale, c.l_window, u->split, u->ns, pstride, \
         h->part_o, h->part_ml
         if (nt == 2) attn_wide_kernel<2><<<u->n, 256, smem, s>>>(HY_WIDE_ARGS);
         else if (nt == 4) attn_wide_kernel<4><<<u->n, 256, smem, s>>>(HY_WIDE_ARGS);
         else attn_wide_kernel<8><<<u->n, 256, smem, s>>>(HY_WIDE_ARGS);
 #undef HY_WIDE_ARGS
-        attn_combine_kernel<WT, float><<<T * H, 64, 0, s>>>(b, h->part_o, h->part_ml, (const WT*)L.sink, nullptr, 0, H, pstride, R,
-                                                            u->split, u->ns, 1.0f, h->f2, h->ld_f2);
+        attn_combine_kernel<WT, float><<<T * H, 64, 0, s>>>(b, h->part_o, h->part_ml, (const WT*)L.sink, nullptr, 0, H, 1, pstride, R,
+                                                            c.l_window, u->split, u->ns, 1.0f, h->f2, h->ld_f2);
         h->launches += 2;
       }
     }
     if (!tc) {
       attn_sink_kernel<AT, WT, float><<<(T * H + 3) / 4, 128, 4 * Dk * sizeof(float), s>>>(
-          b, cv, h->ld_cv, (const AT*)L.cache, (const WT*)L.sink, (const AT*)nullptr, 0, H, 1, Dk, R, c.l_scale, 0.0f, 1, 1.0f,
+          b, cv, h->ld_cv, (const AT*)L.cache, (const WT*)L.sink, (const AT*)nullptr, 0, H, 1, Dk, R, c.l_scale, 0.0f, 1, c.l_window, 1.0f,
           h->f2, h->ld_f2);
       h->launches++;
     }
   }
   {
     ProfScope ps(h, HY_PROF_SMALL_GEMM);
+    const AT* gate = c.l_gate ? pin + L.c_g : nullptr;
     if (T <= 8)
       head_rows_kernel<float, WT, AT><<<(H * dv + 7) / 8, 256, 0, s>>>(T, h->f2, h->ld_f2, R, (const WT*)L.w_uv, H, dv, R, cat,
-                                                                       h->ld_cat, dv);
+                                                                       h->ld_cat, dv, gate, h->ld_pin);
     else
     latent_value_kernel<AT, WT><<<dim3((T + HY_LAT_TB - 1) / HY_LAT_TB, H, (dv + 127) / 128), 128, (size_t)HY_LAT_TB * R * 4, s>>>(
-        T, h->f2, h->ld_f2, (const WT*)L.w_uvT, H, R, dv, cat, h->ld_cat);
+        T, h->f2, h->ld_f2, (const WT*)L.w_uvT, H, R, dv, gate, h->ld_pin, cat, h->ld_cat);
     h->launches++;
   }
 }
@@ -1882,8 +2055,8 @@ int postnorm_layer(hy_engine* h, const Batch& b, size_t li) {
   return HY_OK;
 }
 
-// Routed gated experts over the rows of hb [T, width]: router logits (fp32; with corrected scores they are there already, in
-// h->f1 from column c_router on), the choice with its weights, both products grouped by expert.  Leaves one fp32 row per (token, choice) pair in h->f2 [pairs, width];
+// Routed gated experts over the rows of hb [T, width]: router logits (fp32; a router inside the merged input projection has left
+// them in h->f1 from column c_router on), the choice with its weights, both products grouped by expert.  Leaves one fp32 row per (token, choice) pair in h->f2 [pairs, width];
 // returns whether the rows are in pair order (few pairs) or in the expert-sorted order (h->x_pair_row maps pairs to rows).
 template <typename AT>
 bool routed_gated_experts(hy_engine* h, int T, const AT* hb, const LayerW& L, const hy_layer_cfg& c) {
@@ -1898,8 +2071,9 @@ bool routed_gated_experts(hy_engine* h, int T, const AT* hb, const LayerW& L, co
     ProfScope ps(h, HY_PROF_ROUTE);
     if (c.x_route == HY_ROUTE_CORRECTED_SOFTMAX) {
       const int outputs = NE + c.x_identity;
-      route_corrected_kernel<<<T, 32, (size_t)outputs * 8, s>>>(h->f1 + L.c_router, h->ld_f1, L.x_corr, NE, outputs, top, h->x_ids,
-                                                                h->x_wts, few ? nullptr : h->x_counts);
+      if (L.w_router) gemm<AT, WT, float>(h, hb, W, (const WT*)L.w_router, W, T, outputs, W, to_buf(h->f1, h->ld_f1), L.w_router_t);
+      route_corrected_kernel<<<T, 32, (size_t)(2 * outputs + c.x_groups) * 4, s>>>(h->f1 + L.c_router, h->ld_f1, L.x_corr, NE, outputs, top,
+                                                                                   c.x_groups, c.x_keep, h->x_ids, h->x_wts, few ? nullptr : h->x_counts);
     } else {
       gemm<AT, WT, float>(h, hb, W, (const WT*)L.w_router, W, T, NE, W, to_buf(h->f1, h->ld_f1), L.w_router_t);
       route_top_kernel<<<T, 32, (size_t)NE * 4, s>>>(h->f1, h->ld_f1, nullptr, NE, top, h->x_ids, h->x_wts, few ? nullptr : h->x_counts);
@@ -1977,15 +2151,19 @@ void canon_input(hy_engine* h, const Batch& b, const float* w, float* tails) {
   }
 }
 
+// Attention of a BiasedCfg over the layer's key and value pages: queries in h->pin from column c_q on, result (heads
+// concatenated) in h->cat.
+template <typename AT>
+void biased_attend(hy_engine* h, const Batch& b, const LayerW& L, const hy_layer_cfg& c, const BiasedCfg& bc);
+
 // Biased attention: projections in h->pin (queries, keys, values), result (heads concatenated) in h->cat.
 template <typename AT>
 void biased_mixer(hy_engine* h, const Batch& b, const LayerW& L, const hy_layer_cfg& c) {
-  const int T = b.T, E = b.E;
+  const int T = b.T;
   cudaStream_t s = h->stream;
-  AT* pin = (AT*)h->pin; AT* cat = (AT*)h->cat;
+  AT* pin = (AT*)h->pin;
   const BiasedCfg bc{c.b_heads, c.b_kv_heads, c.b_dim, c.b_vdim, c.b_window, c.b_keep_first, c.b_scale, c.b_softcap, L.b_r1, L.b_r2, L.b_sink,
-                     c.b_chunk, c.b_bias == HY_BIAS_LINEAR ? 1 : 0};
-  const int dp = (c.b_dim <= 64 && c.b_vdim <= 64) ? 64 : 128;
+                     c.b_chunk, c.b_bias, nullptr, 0, 1.0f};
   {
     ProfScope ps(h, HY_PROF_CONV);
     biased_prep_kernel<AT><<<T, 128, 0, s>>>(b, pin, h->ld_pin, L.c_q, c.b_heads * c.b_dim, L.c_k, L.c_v, c.b_kv_heads, c.b_dim, c.b_vdim,
@@ -1993,6 +2171,15 @@ void biased_mixer(hy_engine* h, const Batch& b, const LayerW& L, const hy_layer_
                                              (AT*)h->vfirst, h->ld_vf, (AT*)L.cache, (AT*)L.cache_v);
     h->launches++;
   }
+  biased_attend<AT>(h, b, L, c, bc);
+}
+
+template <typename AT>
+void biased_attend(hy_engine* h, const Batch& b, const LayerW& L, const hy_layer_cfg& c, const BiasedCfg& bc) {
+  const int T = b.T, E = b.E;
+  cudaStream_t s = h->stream;
+  AT* pin = (AT*)h->pin; AT* cat = (AT*)h->cat;
+  const int dp = (c.b_dim <= 64 && c.b_vdim <= 64) ? 64 : 128;
   {
     ProfScope ps(h, HY_PROF_ATTN);
     bool tc = false;
@@ -2016,8 +2203,7 @@ void biased_mixer(hy_engine* h, const Batch& b, const LayerW& L, const hy_layer_
           biased_mma_kernel<128><<<u->n, 128, window_mma_smem(128), s>>>(b, u->d, pin + L.c_q, h->ld_pin, bc, (const bf16*)L.cache,
                                                                               (const bf16*)L.cache_v, cat, h->ld_cat, u->ns, h->part_o, h->part_ml);
         if (u->ns > 1) {
-          biased_combine_kernel<bf16><<<T * c.b_heads, 64, 0, s>>>(h->part_o, h->part_ml, L.b_sink, c.b_heads, c.b_vdim,
-                                                                   dp, u->ns, cat, h->ld_cat);
+          biased_combine_kernel<bf16><<<T * c.b_heads, 64, 0, s>>>(h->part_o, h->part_ml, bc, dp, u->ns, cat, h->ld_cat);
           h->launches++;
         }
       }
@@ -2135,7 +2321,7 @@ void gla_mixer(hy_engine* h, const Batch& b, const LayerW& L, const hy_layer_cfg
     const int async_ok = (dk % ch == 0 && dk % 4 == 0 && dv % ch == 0 && cpb % ch == 0 && h->ld_pin % ch == 0 && L.c_k % ch == 0 && L.c_v % ch == 0) ? 1 : 0;
     cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     kern<<<dim3(H * bph, E), 128, smem, s>>>(b, pin, h->ld_pin, L.c_q, L.c_k, L.c_v, h->f2, h->ld_f2, H, dk, dv, bph, async_ok, L.rec_state,
-                                             h->f2 + c_o, h->ld_f2);
+                                             h->f2 + c_o, h->ld_f2, nullptr, RotPair{0, 1});
   };
   if (dk <= 16) launch(gla_kernel<AT, 16, 4>, 4, gla_smem<AT>(16, 4));
   else if (dk <= 32) launch(gla_kernel<AT, 32, 4>, 4, gla_smem<AT>(32, 4));
@@ -2145,8 +2331,94 @@ void gla_mixer(hy_engine* h, const Batch& b, const LayerW& L, const hy_layer_cfg
   else if (dk <= 512) launch(gla_kernel<AT, 512, 32>, 32, gla_smem<AT>(512, 32));
   else launch(gla_kernel<AT, 1024, 32>, 32, gla_smem<AT>(1024, 32));
   gla_out_kernel<AT><<<(T * H + 3) / 4, 128, 0, s>>>(T, H, dv, h->f2 + c_o, h->ld_f2, pin + L.c_g, h->ld_pin, L.g_norm, h->m.norm_eps,
-                                                     cat, h->ld_cat);
+                                                     1.0f, cat, h->ld_cat);
   h->launches += 2;
+}
+
+// Retention: projections in h->pin (q, k, v, gate); read-outs in h->f2, result in h->cat.
+template <typename AT>
+void retention_mixer(hy_engine* h, const Batch& b, const LayerW& L, const hy_layer_cfg& c) {
+  const int T = b.T, E = b.E, H = c.g_heads, dk = c.g_dim, dv = c.g_vdim;
+  cudaStream_t s = h->stream;
+  AT* pin = (AT*)h->pin; AT* cat = (AT*)h->cat;
+  const RotTable& rot = h->rot_tables[(size_t)L.rot_table].t;
+  const RotPair rp{rot.pairs, c.r_half};
+  ProfScope ps(h, HY_PROF_DELTA);
+  const int ch = 16 / (int)sizeof(AT);
+  auto launch = [&](auto kern, int parts, size_t smem) {
+    const int cpb = 128 / parts, bph = (dv + cpb - 1) / cpb;
+    const int async_ok = (dk % ch == 0 && dv % ch == 0 && cpb % ch == 0 && h->ld_pin % ch == 0 && L.c_k % ch == 0 && L.c_v % ch == 0) ? 1 : 0;
+    cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    kern<<<dim3(H * bph, E), 128, smem, s>>>(b, pin, h->ld_pin, L.c_q, L.c_k, L.c_v, rot.out, rot.ld, H, dk, dv, bph, async_ok, L.rec_state,
+                                             h->f2, h->ld_f2, L.decay, rp);
+  };
+  if (dk <= 16) launch(gla_kernel<AT, 16, 4, true>, 4, gla_smem<AT>(16, 4));
+  else if (dk <= 32) launch(gla_kernel<AT, 32, 4, true>, 4, gla_smem<AT>(32, 4));
+  else if (dk <= 64) launch(gla_kernel<AT, 64, 4, true>, 4, gla_smem<AT>(64, 4));
+  else if (dk <= 128) launch(gla_kernel<AT, 128, 8, true>, 8, gla_smem<AT>(128, 8));
+  else if (dk <= 256) launch(gla_kernel<AT, 256, 16, true>, 16, gla_smem<AT>(256, 16));
+  else if (dk <= 512) launch(gla_kernel<AT, 512, 32, true>, 32, gla_smem<AT>(512, 32));
+  else launch(gla_kernel<AT, 1024, 32, true>, 32, gla_smem<AT>(1024, 32));
+  gla_out_kernel<AT><<<(T * H + 3) / 4, 128, 0, s>>>(T, H, dv, h->f2, h->ld_f2, pin + L.c_g, h->ld_pin, nullptr, h->m.norm_eps, 1.0f, cat,
+                                                     h->ld_cat);
+  h->launches += 2;
+}
+
+// Attention whose values are its unrotated keys beside a gated delta rule with one decay per head: operand columns in h->pin
+// (q, k | convolved q, k, v | gate), fp32 columns in h->f1 (head gates | step sizes | decays); both results in h->cat.
+template <typename AT>
+void attn_delta_mixer(hy_engine* h, const Batch& b, const LayerW& L, const hy_layer_cfg& c) {
+  typedef AT WT;
+  const int T = b.T, E = b.E;
+  cudaStream_t s = h->stream;
+  AT* pin = (AT*)h->pin; AT* cat = (AT*)h->cat; AT* cv = (AT*)h->cv;
+  const RotTable& rot = h->rot_tables[(size_t)L.rot_table].t;
+  const int H = c.d_heads, G = c.d_kv_heads, dk = c.d_dim, dv = c.d_vdim, nk = G * dk, C = 2 * nk + H * dv;
+  {
+    ProfScope ps(h, HY_PROF_CONV);
+    key_value_prep_kernel<AT><<<T, 128, 0, s>>>(b, pin, h->ld_pin, L.c_q, L.c_k, c.b_heads, c.b_kv_heads, c.b_dim, rot.out, rot.ld,
+                                                RotPair{rot.pairs, c.r_half}, (AT*)L.cache, (AT*)L.cache_v);
+    conv_kernel<AT, WT><<<dim3((C + 127) / 128, T), 128, 0, s>>>(b, pin, h->ld_pin, L.c_x, C, c.d_conv, (const WT*)L.conv_qkv,
+                                                                 (const WT*)nullptr, 1, L.conv_state, cv, h->ld_cv);
+    conv_tail_kernel<AT><<<dim3((C + 127) / 128, E), 128, 0, s>>>(b, pin, h->ld_pin, L.c_x, C, c.d_conv, L.conv_state);
+    h->launches += 3;
+  }
+  const BiasedCfg bc{c.b_heads, c.b_kv_heads, c.b_dim, c.b_vdim, 0, 0, c.b_scale, 0.0f, nullptr, nullptr, nullptr, 0, HY_BIAS_NONE,
+                     h->f1, h->ld_f1, c.left_scale};
+  biased_attend<AT>(h, b, L, c, bc);
+  ProfScope ps(h, HY_PROF_DELTA);
+  const int ch = 16 / (int)sizeof(AT);
+  auto launch = [&](auto kern, int parts, size_t smem) {
+    const int cpb = 128 / parts, bph = (dv + cpb - 1) / cpb;
+    const int async_ok = (dk % ch == 0 && dv % ch == 0 && cpb % ch == 0 && h->ld_cv % ch == 0) ? 1 : 0;
+    cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    kern<<<dim3(H * bph, E), 128, smem, s>>>(b, cv, h->ld_cv, 0, nk, 2 * nk, h->f1 + c.b_heads, h->ld_f1, (const float*)L.A_log,
+                                             (const float*)L.dt_bias, H, G, dk, dv, bph, async_ok, L.rec_state, h->f2, h->ld_f2);
+  };
+  if (dk <= 16) launch(delta_head_kernel<AT, 16, 4>, 4, delta_head_smem<AT>(16, 4));
+  else if (dk <= 32) launch(delta_head_kernel<AT, 32, 4>, 4, delta_head_smem<AT>(32, 4));
+  else if (dk <= 64) launch(delta_head_kernel<AT, 64, 4>, 4, delta_head_smem<AT>(64, 4));
+  else if (dk <= 128) launch(delta_head_kernel<AT, 128, 8>, 8, delta_head_smem<AT>(128, 8));
+  else if (dk <= 256) launch(delta_head_kernel<AT, 256, 16>, 16, delta_head_smem<AT>(256, 16));
+  else if (dk <= 512) launch(delta_head_kernel<AT, 512, 32>, 32, delta_head_smem<AT>(512, 32));
+  else launch(delta_head_kernel<AT, 1024, 32>, 32, delta_head_smem<AT>(1024, 32));
+  gla_out_kernel<AT><<<(T * H + 3) / 4, 128, 0, s>>>(T, H, dv, h->f2, h->ld_f2, pin + L.c_g, h->ld_pin, L.g_norm, h->m.norm_eps,
+                                                     c.right_scale, cat + L.o_scan, h->ld_cat);
+  h->launches += 2;
+}
+
+// One row kernel between two sublayers, see RowClose (nothing to do: no launch).
+template <typename AT>
+void launch_row_close(hy_engine* h, int T, RowClose rc) {
+  typedef AT WT;
+  const int W = h->m.width;
+  static bool attr = false;                                  // per AT: this function is a template
+  if (!attr) { cudaFuncSetAttribute(row_close_kernel<AT, WT>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024); attr = true; }
+  rc.eps = h->m.norm_eps;
+  if (!rc.rows && !rc.y && !rc.cast_out && !rc.norm_w) return;
+  ProfScope ps(h, HY_PROF_NORM);
+  row_close_kernel<AT, WT><<<T, 256, (size_t)W * 4, h->stream>>>(rc, W, h->x, (AT*)h->hbuf);
+  h->launches++;
 }
 
 // Between two layer runs: the mixture of a routed feed-forward into the stream (rc.rows NULL: nothing to add), then what run
@@ -2154,19 +2426,48 @@ void gla_mixer(hy_engine* h, const Batch& b, const LayerW& L, const hy_layer_cfg
 // or once that projection has run (projected).
 template <typename AT>
 void close_rows(hy_engine* h, int T, RowClose rc, size_t next, bool projected) {
-  typedef AT WT;
   const int W = h->m.width;
-  static bool attr = false;                                  // per AT: this function is a template
-  if (!attr) { cudaFuncSetAttribute(row_close_kernel<AT, WT>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024); attr = true; }
-  rc.eps = h->m.norm_eps;
   if (next < h->runs.size()) {
     if (h->runs[next].begins && !projected) { rc.cast_out = h->loop_cat; rc.ld_cast = 2 * W; }
     else rc.norm_w = h->lw[next].norm1;
   }
-  if (!rc.rows && !rc.cast_out && !rc.norm_w) return;
-  ProfScope ps(h, HY_PROF_NORM);
-  row_close_kernel<AT, WT><<<T, 256, (size_t)W * 4, h->stream>>>(rc, W, h->x, (AT*)h->hbuf);
-  h->launches++;
+  launch_row_close<AT>(h, T, rc);
+}
+
+// One layer of a norm - sublayer - norm model with plain RMS weights:  x += n1b(mixer(n1 x));  x += n2b(experts(n2 x)).  On entry
+// h->hbuf holds the rows normed by n1, on exit by the next layer's: the norm of a sublayer's result, the residual sum and the
+// norm that the next sublayer reads are one row kernel.
+template <typename AT>
+int rms_sandwich_layer(hy_engine* h, const Batch& b, size_t li) {
+  typedef AT WT;
+  const hy_layer_cfg& c = h->lc[li];
+  const LayerW& L = h->lw[li];
+  const int W = h->m.width, T = b.T;
+  AT* hb = (AT*)h->hbuf; AT* pin = (AT*)h->pin; AT* cat = (AT*)h->cat;
+  {
+    ProfScope ps(h, HY_PROF_GEMM_IN);
+    GemmOut o{};
+    o.out1 = pin; o.ld1 = h->ld_pin; o.split = L.n_mix; o.out2 = h->f1; o.ld2 = h->ld_f1; o.out2_f32 = 1; o.alpha = 1.0f;
+    gemm<AT, WT, AT>(h, hb, W, (const WT*)L.w_in, W, T, L.n_in, W, o, L.w_in_t);
+  }
+  if (c.mixer == HY_MIX_RETENTION) retention_mixer<AT>(h, b, L, c);
+  else if (c.mixer == HY_MIX_ATTN_DELTA) attn_delta_mixer<AT>(h, b, L, c);
+  else latent_mixer<AT>(h, b, L, c);
+  {
+    ProfScope ps(h, HY_PROF_GEMM_OUT);
+    gemm<AT, WT, float>(h, cat, h->ld_cat, (const WT*)L.w_out, L.k_out, T, W, L.k_out, to_buf(h->f2, h->ld_f2), L.w_out_t);
+  }
+  RowClose rc{};
+  rc.y = h->f2; rc.ldy = h->ld_f2; rc.post_w = L.norm1b;
+  if (c.ff_kind == HY_FF_NONE) { close_rows<AT>(h, T, rc, li + 1, false); return HY_OK; }
+  rc.norm_w = L.norm2;
+  launch_row_close<AT>(h, T, rc);
+  const bool few = routed_gated_experts<AT>(h, T, hb, L, c);
+  rc = RowClose{};
+  rc.rows = h->f2; rc.ldr = W; rc.pair_row = few ? nullptr : h->x_pair_row; rc.ids = h->x_ids; rc.wts = h->x_wts;
+  rc.top = c.x_top; rc.n_experts = c.x_experts; rc.post_w = L.norm2b;
+  close_rows<AT>(h, T, rc, li + 1, false);
+  return HY_OK;
 }
 
 // One layer run of a one-norm-per-layer model with plain RMS weights: x += mixer(n(x)) + ff(n(x)).  On entry h->hbuf holds
@@ -2248,6 +2549,10 @@ int run_step(hy_engine* h, const Batch& b, int n_want, const int* want_d, float*
       embed_kernel<WT><<<T, 128, 0, s>>>(b, (const WT*)h->embed, h->inv_freq, h->m.emb_scale, W, h->x);
     }
     h->launches++;
+    if (!h->rot_tables.empty()) {
+      rot_tables_kernel<<<dim3(T, (unsigned)h->rot_tables.size()), 32, 0, s>>>(b, h->rot_tables_d);
+      h->launches++;
+    }
     // output-normed blocks read the stream itself: it leaves here in the activation type too, normed when the model says so
     if (h->m.loop_times > 0) {
       loop_origin_kernel<AT><<<T, 128, 0, s>>>(h->x, W, (AT*)h->loop_cat);
@@ -2256,12 +2561,14 @@ int run_step(hy_engine* h, const Batch& b, int n_want, const int* want_d, float*
     if (h->m.block_kind == HY_BLOCK_POSTNORM) post_norm_add<AT>(h, T, h->x, W, nullptr, nullptr, nullptr, 0, nullptr, h->embed_norm, nullptr, 0);
   }
   const bool rms_parallel = h->m.block_kind == HY_BLOCK_PARALLEL && h->m.norm_kind == HY_NORM_RMS;
-  if (rms_parallel) close_rows<AT>(h, T, RowClose{}, 0, false);
+  const bool rms_sandwich = h->m.block_kind == HY_BLOCK_SANDWICH && h->m.norm_kind == HY_NORM_RMS;
+  if (rms_parallel || rms_sandwich) close_rows<AT>(h, T, RowClose{}, 0, false);
   for (size_t li = 0; li < h->lc.size(); ++li) {
     const hy_layer_cfg& c = h->lc[li];
     const LayerW& L = h->lw[li];
     if (h->m.block_kind != HY_BLOCK_PARALLEL || rms_parallel) {
       if (rms_parallel) parallel_layer<AT>(h, b, li);
+      else if (rms_sandwich) rms_sandwich_layer<AT>(h, b, li);
       else if (h->m.block_kind == HY_BLOCK_SANDWICH) sandwich_layer<AT>(h, b, li);
       else if (h->m.block_kind == HY_BLOCK_POSTNORM) postnorm_layer<AT>(h, b, li);
       else prenorm_layer<AT>(h, b, li);
@@ -2300,20 +2607,20 @@ int run_step(hy_engine* h, const Batch& b, int n_want, const int* want_d, float*
         if ((c.a_dim == 32 || c.a_dim == 64 || c.a_dim == 128) && h->part_o && (u = attn_units(h, E, T, c.a_heads, c.a_kv_heads))) {
           tc = true;
 #define HY_ATTN_ARGS b, u->d, cv, h->ld_cv, (const bf16*)L.cache, c.a_heads, c.a_kv_heads, c.a_scale, c.a_qt_coef, \
-          c.a_qt_every, u->split, u->ns, c.a_dim, h->part_o, h->part_ml
+          c.a_qt_every, 0, u->split, u->ns, c.a_dim, h->part_o, h->part_ml
           if (c.a_dim == 32) attn_mma_kernel<32><<<u->n, 128, 0, s>>>(HY_ATTN_ARGS);
           else if (c.a_dim == 64) attn_mma_kernel<64><<<u->n, 128, 0, s>>>(HY_ATTN_ARGS);
           else attn_mma_kernel<128><<<u->n, 128, 0, s>>>(HY_ATTN_ARGS);
 #undef HY_ATTN_ARGS
           attn_combine_kernel<WT, bf16><<<T * c.a_heads, 64, 0, s>>>(b, h->part_o, h->part_ml, (const WT*)L.sink, pin + L.c_g, h->ld_pin,
-              c.a_heads, c.a_dim, c.a_dim, u->split, u->ns, c.left_scale, cat + L.o_mix, h->ld_cat);
+              c.a_heads, c.a_kv_heads, c.a_dim, c.a_dim, 0, u->split, u->ns, c.left_scale, cat + L.o_mix, h->ld_cat);
           h->launches++;
         }
       }
       if (!tc)
       attn_sink_kernel<AT, WT, AT><<<(T * c.a_heads + 3) / 4, 128, 4 * c.a_dim * sizeof(float), s>>>(
           b, cv, h->ld_cv, (const AT*)L.cache, (const WT*)L.sink, pin + L.c_g, h->ld_pin, c.a_heads, c.a_kv_heads, c.a_dim, c.a_dim,
-          c.a_scale, c.a_qt_coef, c.a_qt_every, c.left_scale, cat + L.o_mix, h->ld_cat);
+          c.a_scale, c.a_qt_coef, c.a_qt_every, 0, c.left_scale, cat + L.o_mix, h->ld_cat);
       }
       h->launches += 4;
       // scan side

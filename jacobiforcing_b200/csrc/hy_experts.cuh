@@ -89,14 +89,16 @@ __global__ void __launch_bounds__(32) route_top_kernel(const float* __restrict__
 }
 
 // A third way: softmax scores s over all `outputs` router outputs (experts, then identity experts), choice by the largest
-// s + correction (ties to the lower index), weights = s of the chosen, not renormalised.  Identity choices (index >= experts)
+// s + correction (ties to the lower index), weights = s of the chosen, not renormalised.  With groups > 1 only outputs of the
+// `keep` groups of neighbouring outputs with the largest single choice score can be chosen.  Identity choices (index >= experts)
 // take no row of the sorted order, so they are not counted.  One warp per token; every choice is a warp-wide maximum.
 __global__ void __launch_bounds__(32) route_corrected_kernel(const float* __restrict__ logits, int ldl, const float* __restrict__ correction,
-                                                             int experts, int outputs, int top, int* __restrict__ ids,
+                                                             int experts, int outputs, int top, int groups, int keep, int* __restrict__ ids,
                                                              float* __restrict__ wts, int* __restrict__ counts) {
   extern __shared__ __align__(16) unsigned char hy_smem[];
   float* s = reinterpret_cast<float*>(hy_smem);                // [outputs] scores
   float* ch = s + outputs;                                     // [outputs] choice scores, -inf once chosen
+  float* gs = ch + outputs;                                    // [groups] largest choice score
   const int t = blockIdx.x, lane = threadIdx.x;
   const float* z = logits + (size_t)t * ldl;
   float mx = -INFINITY;
@@ -107,6 +109,22 @@ __global__ void __launch_bounds__(32) route_corrected_kernel(const float* __rest
   const float inv = 1.0f / warp_sum(sum);
   for (int e = lane; e < outputs; e += 32) { const float v = s[e] * inv; s[e] = v; ch[e] = v + correction[e]; }
   __syncwarp();
+  if (groups > 1) {
+    const int per = outputs / groups;
+    for (int g = lane; g < groups; g += 32) {
+      float m = -INFINITY;
+      for (int i = 0; i < per; ++i) m = fmaxf(m, ch[g * per + i]);
+      gs[g] = m;
+    }
+    __syncwarp();
+    for (int g = lane; g < groups; g += 32) {
+      int better = 0;                                          // groups that come before this one
+      for (int i = 0; i < groups; ++i) better += gs[i] > gs[g] || (gs[i] == gs[g] && i < g);
+      if (better >= keep)
+        for (int i = 0; i < per; ++i) ch[g * per + i] = -INFINITY;
+    }
+    __syncwarp();
+  }
   for (int k = 0; k < top; ++k) {
     float bv = -INFINITY; int best = 0x7fffffff;
     for (int e = lane; e < outputs; e += 32) if (ch[e] > bv) { bv = ch[e]; best = e; }

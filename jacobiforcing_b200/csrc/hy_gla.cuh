@@ -1,15 +1,18 @@
-// hy_gla.cuh — gated linear attention with one decay per key channel, and the row kernels of one-norm-per-layer blocks
-// with plain RMS weights (libjf_hybrid.so).
+// hy_gla.cuh — gated linear attention with one decay per key channel, retention (one fixed decay per head, rotated queries and
+// keys), and the row kernels between the sublayers of blocks with plain RMS weights (libjf_hybrid.so).
 //
 // Per head, S [dim, vdim]:  S <- diag(a) S + k v^T ;  o = S^T q dim^(-1/2)   (the read-out sees the current token's write)
 //   out = o / rms(o) * norm_w * silu(g)        (norm over the head's vdim, one weight shared by the heads)
-// The decay a = sigmoid(z)^(1 / tau) leaves the decay projection's epilogue as fp32 (gemm_store).
+// The decay a = sigmoid(z)^(1 / tau) leaves the decay projection's epilogue as fp32 (gemm_store).  Retention is the same
+// recurrence with one number per head for a and with q, k rotated at their position (in fp32, between the projections and the
+// recurrence) and no weight in the norm.
 //
 // The recurrence has no feedback from the read-out and its value columns are independent, so a head is cut into blocks of
 // CPB = 128 / PARTS columns that run side by side on different SMs, and PARTS lanes share a column, each holding DR / PARTS
 // of its key rows in registers.  The norm needs whole heads: it follows in a kernel of its own (gla_out_kernel).
 #pragma once
 #include "hy_kernels.cuh"
+#include "hy_delta.cuh"
 #include "jf_ptx.cuh"
 
 namespace hy {
@@ -29,17 +32,19 @@ __host__ __device__ constexpr size_t gla_smem(int dr, int parts) {
 // 4 (r + PARTS i) .. + 3, so the PARTS row quadruples a warp reads from shared memory at once lie next to each other.
 // async_ok: head sizes, leading dimensions and column offsets are multiples of 16 bytes, and so is CPB: raw rows of the next batch of tokens travel by asynchronous
 // copies while the current batch runs; short entries (decode steps) and odd sizes stage directly.
-template <typename AT, int DR, int PARTS>
+// ROT (retention): `decay` holds the cosines and sines of the step's positions instead (rot_tables_kernel; the first 2 pairs
+// dimensions rotate as `rp` says), head_decay [H] the decays.
+template <typename AT, int DR, int PARTS, bool ROT = false>
 __global__ void __launch_bounds__(128) gla_kernel(Batch b, const AT* __restrict__ in, int ld, int col_q, int col_k, int col_v,
                                                   const float* __restrict__ decay, int ldd, int H, int dim, int vdim,
                                                   int blocks_per_head, int async_ok, float* __restrict__ state,
-                                                  float* __restrict__ o, int ldo) {
+                                                  float* __restrict__ o, int ldo, const float* __restrict__ head_decay, RotPair rp) {
   constexpr int TB = gla_tb(DR), RP = DR / PARTS, CW = 32 / PARTS, CPB = 4 * CW, CH = 16 / (int)sizeof(AT);
   extern __shared__ __align__(16) unsigned char hy_smem[];
   float* sq = reinterpret_cast<float*>(hy_smem);               // [TB][DR] scaled queries
   float* sk = sq + TB * DR;                                    // [TB][DR] keys
   float* sv = sk + TB * DR;                                    // [TB][CPB] values
-  float* sa = sv + TB * CPB;                                   // [2][TB][DR] decays (used in place)
+  float* sa = sv + TB * CPB;                                   // [2][TB][DR] decays (used in place), or cosines | sines
   constexpr int RW = 2 * DR + (CPB < 8 ? 8 : CPB);
   AT* raw = reinterpret_cast<AT*>(sa + 2 * TB * DR);           // [2][TB][RW] raw q | k | v rows in flight
   const int h = blockIdx.x / blocks_per_head, c0 = (blockIdx.x % blocks_per_head) * CPB, e = blockIdx.y;
@@ -60,7 +65,9 @@ __global__ void __launch_bounds__(128) gla_kernel(Batch b, const AT* __restrict_
   const AT* inq = in + col_q + h * dim;
   const AT* ink = in + col_k + h * dim;
   const AT* inv = in + col_v + h * vdim + c0;
-  const float* dec = decay + h * dim;
+  const float* dec = decay + (ROT ? 0 : h * dim);
+  const int ndec = ROT ? 2 * rp.pairs : dim;                   // floats of a token's row of `decay` that are used
+  const float hd = ROT ? head_decay[h] : 0.0f;
   // copies of a batch's raw rows: 16 bytes at a time, the row pitches are compile-time so no division by a run-time size
   auto fetch = [&](int j0, int nb, int buf) {
     AT* dst = raw + (size_t)buf * TB * RW;
@@ -75,7 +82,7 @@ __global__ void __launch_bounds__(128) gla_kernel(Batch b, const AT* __restrict_
     }
     for (int i = tid; i < nb * AC; i += 128) {
       const int tt = i / AC, k = i % AC * 4;
-      if (k < dim) jf::cp_async_16(da + (size_t)tt * DR + k, dec + (t0 + tt) * ldd + k, 16u);
+      if (k < ndec) jf::cp_async_16(da + (size_t)tt * DR + k, dec + (t0 + tt) * ldd + k, 16u);
     }
     for (int i = tid; i < nb * VC; i += 128) {
       const int tt = i / VC, k = i % VC * CH;
@@ -85,7 +92,8 @@ __global__ void __launch_bounds__(128) gla_kernel(Batch b, const AT* __restrict_
   };
   if (ahead) {
     // rows beyond the head's key size are never copied: q and k are zero there, so the decay only has to be a number
-    for (int i = tid; i < 2 * TB * DR; i += 128) if (i % DR >= dim) sa[i] = 0.0f;
+    if (!ROT)
+      for (int i = tid; i < 2 * TB * DR; i += 128) if (i % DR >= dim) sa[i] = 0.0f;
     fetch(0, min(TB, cnt), 0);
   }
   // one token's update of this lane's key rows; returns its part of the read-out
@@ -97,7 +105,8 @@ __global__ void __launch_bounds__(128) gla_kernel(Batch b, const AT* __restrict_
     float p0 = 0.0f, p1 = 0.0f, p2 = 0.0f, p3 = 0.0f;
 #pragma unroll
     for (int i = 0; i < RP / 4; ++i) {
-      const float4 a = a4[i * PARTS], k = k4[i * PARTS], q = q4[i * PARTS];
+      const float4 k = k4[i * PARTS], q = q4[i * PARTS];
+      const float4 a = ROT ? make_float4(hd, hd, hd, hd) : a4[i * PARTS];
       S[4 * i] = fmaf(a.x, S[4 * i], k.x * v);         p0 = fmaf(S[4 * i], q.x, p0);
       S[4 * i + 1] = fmaf(a.y, S[4 * i + 1], k.y * v); p1 = fmaf(S[4 * i + 1], q.y, p1);
       S[4 * i + 2] = fmaf(a.z, S[4 * i + 2], k.z * v); p2 = fmaf(S[4 * i + 2], q.z, p2);
@@ -122,6 +131,38 @@ __global__ void __launch_bounds__(128) gla_kernel(Batch b, const AT* __restrict_
           rq = *reinterpret_cast<const VecN<AT, CH>*>(src + (size_t)tt * RW + k);
           rk = *reinterpret_cast<const VecN<AT, CH>*>(src + (size_t)tt * RW + DR + k);
         }
+        if (ROT && k < ndec) {
+          const float* cs = ca + (size_t)tt * DR;
+          float fq[CH], fk[CH];
+          if (rp.half && rp.pairs % CH == 0) {                 // the partners of a chunk are a chunk
+            const bool hi = k >= rp.pairs;
+            const int kp = hi ? k - rp.pairs : k + rp.pairs, p0 = hi ? kp : k;
+            const VecN<AT, CH> wq = *reinterpret_cast<const VecN<AT, CH>*>(src + (size_t)tt * RW + kp);
+            const VecN<AT, CH> wk = *reinterpret_cast<const VecN<AT, CH>*>(src + (size_t)tt * RW + DR + kp);
+#pragma unroll
+            for (int c = 0; c < CH; ++c) {
+              const float co = cs[p0 + c], si = hi ? cs[rp.pairs + p0 + c] : -cs[rp.pairs + p0 + c];
+              fq[c] = fmaf(to_f(rq.v[c]), co, to_f(wq.v[c]) * si);
+              fk[c] = fmaf(to_f(rk.v[c]), co, to_f(wk.v[c]) * si);
+            }
+          } else {
+#pragma unroll
+            for (int c = 0; c < CH; ++c) {
+              fq[c] = to_f(rq.v[c]); fk[c] = to_f(rk.v[c]);
+              if (k + c < ndec) {
+                const int kp = rp.partner(k + c);
+                fq[c] = rp.turn(cs, k + c, fq[c], to_f(src[(size_t)tt * RW + kp]));
+                fk[c] = rp.turn(cs, k + c, fk[c], to_f(src[(size_t)tt * RW + DR + kp]));
+              }
+            }
+          }
+#pragma unroll
+          for (int c = 0; c < CH; c += 4) {
+            *reinterpret_cast<float4*>(&sq[tt * DR + k + c]) = make_float4(fq[c] * qscale, fq[c + 1] * qscale, fq[c + 2] * qscale, fq[c + 3] * qscale);
+            *reinterpret_cast<float4*>(&sk[tt * DR + k + c]) = make_float4(fk[c], fk[c + 1], fk[c + 2], fk[c + 3]);
+          }
+          continue;
+        }
 #pragma unroll
         for (int c = 0; c < CH; c += 4) {
           *reinterpret_cast<float4*>(&sq[tt * DR + k + c]) = make_float4(to_f(rq.v[c]) * qscale, to_f(rq.v[c + 1]) * qscale, to_f(rq.v[c + 2]) * qscale, to_f(rq.v[c + 3]) * qscale);
@@ -137,9 +178,18 @@ __global__ void __launch_bounds__(128) gla_kernel(Batch b, const AT* __restrict_
         const int tt = i / DR, k = i % DR;
         const size_t t = (size_t)(start + j0 + tt);
         const bool ok = k < dim;
-        sq[i] = ok ? to_f(inq[t * ld + k]) * qscale : 0.0f;
-        sk[i] = ok ? to_f(ink[t * ld + k]) : 0.0f;
-        ca[i] = ok ? dec[t * ldd + k] : 0.0f;
+        float q = ok ? to_f(inq[t * ld + k]) : 0.0f, kk = ok ? to_f(ink[t * ld + k]) : 0.0f;
+        if (ROT) {
+          if (k < ndec) {
+            const int kp = rp.partner(k);
+            q = rp.turn(dec + t * ldd, k, q, to_f(inq[t * ld + kp]));
+            kk = rp.turn(dec + t * ldd, k, kk, to_f(ink[t * ld + kp]));
+          }
+        } else {
+          ca[i] = ok ? dec[t * ldd + k] : 0.0f;
+        }
+        sq[i] = q * qscale;
+        sk[i] = kk;
       }
       for (int i = tid; i < nb * CPB; i += 128) {
         const int tt = i / CPB, k = i % CPB;
@@ -194,31 +244,33 @@ __global__ void __launch_bounds__(128) gla_kernel(Batch b, const AT* __restrict_
   }
 }
 
-// Norm per head, weight, output gate: out[t, h, :] = o / rms(o) * w * silu(g).  One warp per (token, head).
+// Norm per head, weight (NULL: none), output gate: out[t, h, :] = o / rms(o) * w * silu(g) * out_scale.  One warp per (token, head).
 template <typename AT>
 __global__ void __launch_bounds__(128) gla_out_kernel(int T, int H, int vdim, const float* __restrict__ o, int ldi,
                                                       const AT* __restrict__ g, int ldg, const float* __restrict__ w, float eps,
-                                                      AT* __restrict__ out, int ldo) {
+                                                      float out_scale, AT* __restrict__ out, int ldo) {
   const int unit = blockIdx.x * 4 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
   if (unit >= T * H) return;
   const size_t t = unit / H, c0 = (size_t)(unit % H) * vdim;
   const float* orow = o + t * ldi + c0;
   float ss = 0.0f;
   for (int k = lane; k < vdim; k += 32) ss = fmaf(orow[k], orow[k], ss);
-  const float inv = 1.0f / sqrtf(warp_sum(ss) / (float)vdim + eps);
+  const float inv = out_scale / sqrtf(warp_sum(ss) / (float)vdim + eps);
   for (int k = lane; k < vdim; k += 32)
-    out[t * ldo + c0 + k] = from_f<AT>(orow[k] * inv * w[k] * silu_f(to_f(g[t * ldg + c0 + k])));
+    out[t * ldo + c0 + k] = from_f<AT>(orow[k] * inv * (w ? w[k] : 1.0f) * silu_f(to_f(g[t * ldg + c0 + k])));
 }
 
-// ---- one token's row between two layers of a one-norm-per-layer block -------------------------------------------------------
-// x += the mixture of a routed feed-forward (rows NULL: nothing added), then what the next layer reads: the RMS norm of the
-// row (norm_w), or the row itself (cast_out: the stream's half of the loop projection's operand), in the activation type.
+// ---- one token's row between two sublayers ----------------------------------------------------------------------------------
+// x += a sublayer's result: its rows (y), or the mixture of a routed feed-forward (rows), or nothing (both NULL); through an
+// RMS norm of its own first when post_w is given.  Then what the next sublayer reads: the RMS norm of the row (norm_w), or
+// the row itself (cast_out: the stream's half of the loop projection's operand), in the activation type.
 // A choice >= n_experts stands for the sublayer's input: h [T, width] in the activation type, the buffer the norm is then
 // written to (a thread reads a channel before it writes it).
 struct RowClose {
   const float* rows; int ldr; const int* pair_row; const int* ids; const float* wts; int top, n_experts;
   const void* norm_w; float eps;
   void* cast_out; int ld_cast;
+  const float* y; int ldy; const void* post_w;
 };
 
 template <typename AT, typename WT>
@@ -228,17 +280,27 @@ __global__ void __launch_bounds__(256) row_close_kernel(RowClose c, int width, f
   __shared__ float red[33];
   const int t = blockIdx.x;
   float ss = 0.0f;
+  auto result = [&](int ch) {
+    if (c.y) return c.y[(size_t)t * c.ldy + ch];
+    float y = 0.0f;
+    for (int k = 0; k < c.top; ++k) {
+      const int i = t * c.top + k;
+      const float r = c.ids[i] >= c.n_experts ? to_f(h[(size_t)t * width + ch])
+                                              : c.rows[(size_t)(c.pair_row ? c.pair_row[i] : i) * c.ldr + ch];
+      y = fmaf(c.wts[i], r, y);
+    }
+    return y;
+  };
+  float pinv = 1.0f;
+  if (c.post_w) {
+    for (int ch = threadIdx.x; ch < width; ch += blockDim.x) { const float y = result(ch); xs[ch] = y; ss = fmaf(y, y, ss); }
+    pinv = 1.0f / sqrtf(block_sum(ss, red) / (float)width + c.eps);
+    ss = 0.0f;
+  }
   for (int ch = threadIdx.x; ch < width; ch += blockDim.x) {
     float v = x[(size_t)t * width + ch];
-    if (c.rows) {
-      float y = 0.0f;
-      for (int k = 0; k < c.top; ++k) {
-        const int i = t * c.top + k;
-        const float r = c.ids[i] >= c.n_experts ? to_f(h[(size_t)t * width + ch])
-                                                : c.rows[(size_t)(c.pair_row ? c.pair_row[i] : i) * c.ldr + ch];
-        y = fmaf(c.wts[i], r, y);
-      }
-      v += y;
+    if (c.rows || c.y) {
+      v += c.post_w ? xs[ch] * pinv * to_f(((const WT*)c.post_w)[ch]) : result(ch);
       x[(size_t)t * width + ch] = v;
     }
     xs[ch] = v;

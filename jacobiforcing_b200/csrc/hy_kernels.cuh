@@ -414,19 +414,23 @@ __global__ void cache_append_kernel(Batch b, const AT* __restrict__ k, int ldk, 
   }
 }
 
+// first position that the query at p sees through a sliding window (0: no window)
+__host__ __device__ __forceinline__ int first_seen(int p, int window) { return window > 0 && p - window + 1 > 0 ? p - window + 1 : 0; }
+
 // ---- causal softmax attention with a sink; values are the keys -----------------------------------------------------------------
 // One warp per (token, query head).  Keys are walked in groups of 32 aligned to absolute positions; the running maximum
 // starts at the sink logit and the denominator at exp(sink - sink) = 1: the sink has no key and no value (sink NULL: an
 // ordinary softmax).  The query is
 // multiplied by its position's temperature in fp32.  The value of a key is its first vdim dimensions (vdim == dim: the
-// values are the keys; vdim < dim: a latent followed by a part that only enters the score).  Output: heads concatenated
+// values are the keys; vdim < dim: a latent followed by a part that only enters the score).  window > 0: only the keys j with
+// pos - j < window.  Output: heads concatenated
 // [H, vdim], times sigmoid(gate) when there is a gate, times out_scale.
 constexpr int HY_ATT_MAXD = 20;     // dims per lane: dim <= 640
 template <typename AT, typename WT, typename OT>
 __global__ void __launch_bounds__(128) attn_sink_kernel(Batch b, const AT* __restrict__ q, int ldq, const AT* __restrict__ cache,
                                                         const WT* __restrict__ sink, const AT* __restrict__ gate, int ldg,
                                                         int H, int G, int dim, int vdim, float scale, float qt_coef,
-                                                        int qt_every, float out_scale, OT* __restrict__ out, int ldo) {
+                                                        int qt_every, int window, float out_scale, OT* __restrict__ out, int ldo) {
   extern __shared__ __align__(16) unsigned char hy_smem[];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   float* qs = reinterpret_cast<float*>(hy_smem) + warp * dim;
@@ -443,11 +447,13 @@ __global__ void __launch_bounds__(128) attn_sink_kernel(Batch b, const AT* __res
   float acc[HY_ATT_MAXD];
 #pragma unroll
   for (int i = 0; i < HY_ATT_MAXD; ++i) acc[i] = 0.0f;
-  for (int j0 = 0; j0 <= pos; j0 += 32) {
+  const int first = first_seen(pos, window);
+  for (int j0 = first / 32 * 32; j0 <= pos; j0 += 32) {
     const int j = j0 + lane;
+    const bool sees = j <= pos && j >= first;
     float s = -INFINITY;
     const AT* kr = nullptr;
-    if (j <= pos) {
+    if (sees) {
       kr = cache + (((size_t)pg[j / b.page_size] * G + g) * b.page_size + j % b.page_size) * dim;
       float dot = 0.0f;
       for (int d = 0; d < dim; ++d) dot = fmaf(qs[d], to_f(kr[d]), dot);
@@ -455,13 +461,13 @@ __global__ void __launch_bounds__(128) attn_sink_kernel(Batch b, const AT* __res
     }
     const float mn = fmaxf(m, warp_max(s));
     const float corr = expf(m - mn);
-    const float p = (j <= pos) ? expf(s - mn) : 0.0f;
+    const float p = sees ? expf(s - mn) : 0.0f;
     l = l * corr + warp_sum(p);
     m = mn;
 #pragma unroll
     for (int i = 0; i < HY_ATT_MAXD; ++i) acc[i] *= corr;
     const int cnt = min(32, pos + 1 - j0);
-    for (int jj = 0; jj < cnt; ++jj) {
+    for (int jj = max(first - j0, 0); jj < cnt; ++jj) {
       const float pj = __shfl_sync(0xffffffffu, p, jj);
       const int ja = j0 + jj;
       const AT* kj = cache + (((size_t)pg[ja / b.page_size] * G + g) * b.page_size + ja % b.page_size) * dim;

@@ -278,10 +278,12 @@ __global__ void __launch_bounds__(128) latent_query_kernel(Batch b, const AT* __
 }
 
 // The value up-projection behind the weighted sum: out[t, h, j] = sum_r w_uvT[h][r][j] o[t, h, r]  (o fp32: the weighted
-// sum of latents; w_uvT is the value up-projection transposed per head at load so that thread j reads coalesced).
+// sum of latents; w_uvT is the value up-projection transposed per head at load so that thread j reads coalesced).  gate (NULL: none):
+// the result times sigmoid(gate[t, h * vdim + j]).
 template <typename AT, typename WT>
 __global__ void __launch_bounds__(128) latent_value_kernel(int T, const float* __restrict__ o, int ldi, const WT* __restrict__ w_uvT,
-                                                           int H, int rank, int vdim, AT* __restrict__ out, int ldo) {
+                                                           int H, int rank, int vdim, const AT* __restrict__ gate, int ldg,
+                                                           AT* __restrict__ out, int ldo) {
   extern __shared__ __align__(16) unsigned char hy_smem[];
   float* os = reinterpret_cast<float*>(hy_smem);              // [TB][rank]
   const int t0 = blockIdx.x * HY_LAT_TB, h = blockIdx.y, nb = min(HY_LAT_TB, T - t0);
@@ -301,15 +303,20 @@ __global__ void __launch_bounds__(128) latent_value_kernel(int T, const float* _
 #pragma unroll
     for (int tt = 0; tt < HY_LAT_TB; ++tt) acc[tt] = fmaf(os[tt * rank + k], w, acc[tt]);
   }
-  for (int tt = 0; tt < nb; ++tt) out[(size_t)(t0 + tt) * ldo + h * vdim + j] = from_f<AT>(acc[tt]);
+  for (int tt = 0; tt < nb; ++tt) {
+    const float gt = gate ? sigmoid_f(to_f(gate[(size_t)(t0 + tt) * ldg + h * vdim + j])) : 1.0f;
+    out[(size_t)(t0 + tt) * ldo + h * vdim + j] = from_f<AT>(acc[tt] * gt);
+  }
 }
 
 // Few rows (decode steps): out[t, h, n] = sum_k in[t, h, k] w[h][n][k] for up to 8 rows t.  One warp per (h, n) walks a
 // weight row 16 bytes per lane (both per-head projections around the attention are stored [n][k] for this kernel as well),
-// so the weights stream once at full width instead of one block per head walking them column by column.
+// so the weights stream once at full width instead of one block per head walking them column by column.  gate (NULL: none): the
+// result times sigmoid(gate[t, h * N + n]).
 template <typename TI, typename TW, typename TO>
 __global__ void __launch_bounds__(256) head_rows_kernel(int T, const TI* __restrict__ in, int ldi, int in_hs, const TW* __restrict__ w,
-                                                        int H, int N, int K, TO* __restrict__ out, int ldo, int out_hs) {
+                                                        int H, int N, int K, TO* __restrict__ out, int ldo, int out_hs,
+                                                        const TO* __restrict__ gate = nullptr, int ldg = 0) {
   constexpr int VEC = 16 / sizeof(TW);
   const int lane = threadIdx.x & 31;
   const int id = blockIdx.x * 8 + (threadIdx.x >> 5);
@@ -342,7 +349,10 @@ __global__ void __launch_bounds__(256) head_rows_kernel(int T, const TI* __restr
   for (int t = 0; t < 8; ++t) {
     if (t >= T) break;
     const float v = warp_sum(acc[t]);
-    if (lane == 0) out[(size_t)t * ldo + h * out_hs + n] = from_f<TO>(v);
+    if (lane == 0) {
+      const float gt = gate ? sigmoid_f(to_f(gate[(size_t)t * ldg + h * N + n])) : 1.0f;
+      out[(size_t)t * ldo + h * out_hs + n] = from_f<TO>(v * gt);
+    }
   }
 }
 

@@ -33,6 +33,12 @@ to the softmax's denominator), "latent_attention" (full-rank queries, rotation o
 Feed-forward "dense" (gated, tanh-gelu) or "moe" (clamped gated experts and identity experts, chosen by softmax scores plus
 a correction, weighted by the plain scores).
 
+Architecture "Mafalorn": an RMS norm with a plain weight on both sides of every sublayer.  Mixers: "retention" (linear attention
+with one fixed decay per head, rotated queries and keys), "parallel" (softmax attention whose values are its unrotated keys,
+one output gate per head, beside a gated delta rule with one decay per head), "latent_attention" (full-rank queries, rotated
+neighbours, sliding window, element-wise output gate).  Feed-forward "moe" (gated silu experts and identity experts, chosen
+inside the best groups by softmax scores plus a correction, weighted by the plain scores).
+
 Every size and every constant that can differ between models is read from config.json; sizes that only the tensors know
 (the inner sizes of the two-step decay and gate projections) are read from the checkpoint's tensor shapes."""
 from __future__ import annotations
@@ -46,10 +52,11 @@ from typing import Dict, List, Optional, Tuple
 import numpy as np
 
 MIX_ATTN_SCAN, MIX_DELTA, MIX_SSD, MIX_LATENT, MIX_GLR, MIX_WINDOW, MIX_MLSTM, MIX_BIASED, MIX_GLA = 0, 1, 2, 3, 4, 5, 6, 7, 8
+MIX_RETENTION, MIX_ATTN_DELTA = 9, 10
 FF_NONE, FF_RELU2, FF_ROUTED, FF_GATED = 0, 1, 2, 3
 ACT_SILU, ACT_GELU_TANH, ACT_GELU_ERF, ACT_CLAMPED = 0, 1, 2, 3
 ROUTE_SIGMOID_GROUPS, ROUTE_TOP_SOFTMAX, ROUTE_CORRECTED_SOFTMAX = 0, 1, 2
-BIAS_LOG, BIAS_LINEAR = 0, 1
+BIAS_LOG, BIAS_LINEAR, BIAS_NONE = 0, 1, 2
 NORM_RMS_OFFSET, NORM_TANH, NORM_RMS = 0, 1, 2
 BLOCK_PARALLEL, BLOCK_SANDWICH, BLOCK_POSTNORM, BLOCK_PRENORM = 0, 1, 2, 3
 POS_SINUSOID, POS_NONE = 0, 1
@@ -160,6 +167,11 @@ class LayerSpec:
     g_low: int = 0
     g_tau: float = 1.0
     x_identity: int = 0
+    # latent attention: sliding window (0: none), element-wise output gate
+    l_window: int = 0
+    l_gate: int = 0
+    # fixed decay per head (retention); travels as the fp32 tensor "l<i>.mix.decay"
+    decay: Tuple[float, ...] = ()
 
     def cache_elems_per_token(self) -> int:
         """Elements this layer keeps in the paged cache for every token of a request."""
@@ -169,7 +181,7 @@ class LayerSpec:
             return self.l_kv_rank + self.l_rot_dim
         if self.mixer == MIX_WINDOW:                  # keys and values, and their pooled blocks
             return -(-self.w_kv_heads * (self.w_dim + self.w_vdim) * (self.w_pool + 1) // self.w_pool)
-        if self.mixer == MIX_BIASED:
+        if self.mixer in (MIX_BIASED, MIX_ATTN_DELTA):
             return self.b_kv_heads * (self.b_dim + self.b_vdim)
         return 0
 
@@ -310,6 +322,72 @@ def _clamped_experts_ff(spec: LayerSpec, mlp: dict) -> None:
         raise ValueError("mixture of experts: top must lie in 1..experts + identity")
 
 
+def _rotation(spec: LayerSpec, rot: dict, most: int, what: str) -> None:
+    """rot: dims, base and, when the frequencies are interpolated, scaling (factor, original, fast, slow)."""
+    spec.r_dims, spec.r_base = int(rot["dims"]), float(rot["base"])
+    sc = rot.get("scaling")
+    if sc:
+        spec.r_factor, spec.r_original = float(sc["factor"]), float(sc["original"])
+        spec.r_fast, spec.r_slow = float(sc["fast"]), float(sc["slow"])
+        if min(spec.r_factor, spec.r_original, spec.r_fast, spec.r_slow) <= 0.0:
+            raise ValueError(f"{what}: rot.scaling's numbers must be positive")
+    if spec.r_dims % 2 or not 0 <= spec.r_dims <= most:
+        raise ValueError(f"{what}: rot.dims must be even and at most {most}")
+
+
+def _retention_spec(m: dict) -> LayerSpec:
+    spec = LayerSpec(MIX_RETENTION, g_heads=int(m["heads"]), g_dim=int(m["dim"]), g_vdim=int(m["vdim"]), r_half=1,
+                     decay=tuple(float(x) for x in m["decay"]))
+    if min(spec.g_heads, spec.g_dim, spec.g_vdim) <= 0:
+        raise ValueError("retention: heads, dim and vdim must be positive")
+    if len(spec.decay) != spec.g_heads:
+        raise ValueError("retention: one decay per head")
+    _rotation(spec, m["rot"], spec.g_dim, "retention")
+    return spec
+
+
+def _attn_delta_spec(m: dict) -> LayerSpec:
+    a, d = m["left"], m["right"]
+    spec = LayerSpec(MIX_ATTN_DELTA, b_heads=int(a["heads"]), b_kv_heads=int(a["kv_heads"]), b_dim=int(a["dim"]), b_vdim=int(a["vdim"]),
+                     b_scale=float(a["scale"]), b_bias=BIAS_NONE, b_no_bias=1, r_half=1, d_heads=int(d["heads"]),
+                     d_kv_heads=int(d["kv_heads"]), d_dim=int(d["dim"]), d_vdim=int(d["vdim"]), d_conv=int(d["conv"]),
+                     left_scale=float(m["left_scale"]), right_scale=float(m["right_scale"]))
+    if spec.b_heads <= 0 or spec.b_kv_heads <= 0 or spec.b_heads % spec.b_kv_heads:
+        raise ValueError("parallel, left: heads must be a positive multiple of kv_heads")
+    if spec.b_dim <= 0 or spec.b_vdim != spec.b_dim:
+        raise ValueError("parallel, left: the values are the keys, so vdim must equal dim")
+    if spec.d_heads <= 0 or spec.d_kv_heads <= 0 or spec.d_heads % spec.d_kv_heads:
+        raise ValueError("parallel, right: heads must be a positive multiple of kv_heads")
+    if min(spec.d_dim, spec.d_vdim) <= 0 or not 1 <= spec.d_conv <= 16:
+        raise ValueError("parallel, right: dim and vdim must be positive, conv taps in 1..16")
+    _rotation(spec, a["rot"], spec.b_dim, "parallel, left")
+    return spec
+
+
+def _gated_window_latent_spec(m: dict) -> LayerSpec:
+    spec = LayerSpec(MIX_LATENT, l_heads=int(m["heads"]), l_dim=int(m["dim"]), l_rot_dim=int(m["rot_dim"]), l_vdim=int(m["vdim"]),
+                     l_kv_rank=int(m["kv_rank"]), l_q_rank=0, l_scale=float(m["scale"]), l_no_sink=1, r_half=0,
+                     l_window=int((m.get("mask") or {}).get("size") or 0), l_gate=1)
+    if min(spec.l_heads, spec.l_dim, spec.l_vdim, spec.l_kv_rank) <= 0 or spec.l_window < 0:
+        raise ValueError("latent_attention: sizes must be positive, the window not negative")
+    _rotation(spec, m["rot"], spec.l_rot_dim, "latent_attention")
+    return spec
+
+
+def _grouped_experts_ff(spec: LayerSpec, mlp: dict) -> None:
+    r = mlp["router"]
+    spec.ff_kind, spec.ff = FF_ROUTED, int(mlp["expert"]["ff"])
+    spec.x_experts, spec.x_top, spec.x_identity = int(r["experts"]), int(r["top"]), int(r.get("identity") or 0)
+    spec.x_route, spec.x_plain, spec.x_act = ROUTE_CORRECTED_SOFTMAX, 0, ACT_SILU
+    g = r.get("groups") or {"count": 1, "keep": 1}
+    spec.x_groups, spec.x_keep = int(g["count"]), int(g["keep"])
+    outputs = spec.x_experts + spec.x_identity
+    if spec.x_identity < 0 or spec.x_groups <= 0 or outputs % spec.x_groups or not 1 <= spec.x_keep <= spec.x_groups:
+        raise ValueError("mixture of experts: experts + identity must split into groups.count equal groups, 1 <= keep <= count")
+    if not 1 <= spec.x_top <= spec.x_keep * (outputs // spec.x_groups):
+        raise ValueError("mixture of experts: top exceeds the outputs a token may choose from")
+
+
 @dataclass
 class HybridConfig:
     architecture: str
@@ -361,6 +439,8 @@ class HybridConfig:
             return cls._sebavik(cfg)
         if cfg.get("architecture") == "Kisadra":
             return cls._kisadra(cfg, shapes)
+        if cfg.get("architecture") == "Mafalorn":
+            return cls._mafalorn(cfg)
         layers = []
         for i, lc in enumerate(cfg["layers"]):
             m = lc["mixer"]
@@ -502,6 +582,24 @@ class HybridConfig:
             if not 0 <= hc.loop_start < hc.loop_stop <= len(layers) or hc.loop_times < 1:
                 raise ValueError("loop: 0 <= start < stop <= number of layers, times at least 1")
         return hc
+
+    @classmethod
+    def _mafalorn(cls, cfg: dict) -> "HybridConfig":
+        layers: List[LayerSpec] = []
+        specs = {"retention": _retention_spec, "parallel": _attn_delta_spec, "latent_attention": _gated_window_latent_spec}
+        for lc in cfg["layers"]:
+            if lc["type"] not in specs:
+                raise NotImplementedError(f"layer type {lc['type']!r}")
+            spec = specs[lc["type"]](lc["mixer"])
+            mlp = lc.get("mlp")
+            if mlp is not None:
+                if mlp.get("kind") != "moe":
+                    raise NotImplementedError(f"feed-forward kind {mlp.get('kind')!r}")
+                _grouped_experts_ff(spec, mlp)
+            layers.append(spec)
+        return cls(architecture="Mafalorn", width=int(cfg["width"]), vocab=int(cfg["vocab"]), emb_scale=1.0,
+                   logit_scale=float(cfg.get("logit_scale", 1.0)), norm_eps=float(cfg["norm"]["eps"]), layers=layers,
+                   norm_kind=NORM_RMS, block_kind=BLOCK_SANDWICH, pos_kind=POS_NONE)
 
     @classmethod
     def from_dir(cls, path: str) -> "HybridConfig":

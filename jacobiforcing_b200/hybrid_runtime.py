@@ -103,6 +103,9 @@ class HybridRuntime:
         self.finalize()
 
     def finalize(self) -> None:
+        for i, s in enumerate(self.config.layers):                     # constants of the configuration that are one number per head
+            if s.decay:
+                self.load_tensor(f"l{i}.mix.decay", 1, [len(s.decay)], np.asarray(s.decay, dtype=np.float32))
         cabi.check(self.lib.hy_finalize(self.h), self.h)
 
     # ---- one step ---------------------------------------------------------------------------------------------------

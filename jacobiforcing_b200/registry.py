@@ -43,6 +43,7 @@ FAMILIES: Dict[str, ModelFamily] = {
     "Vosolorn": ModelFamily("hybrid", True, _hybrid_config, _hybrid_runner),
     "Sebavik": ModelFamily("hybrid", True, _hybrid_config, _hybrid_runner),
     "Kisadra": ModelFamily("hybrid", True, _hybrid_config, _hybrid_runner),
+    "Mafalorn": ModelFamily("hybrid", True, _hybrid_config, _hybrid_runner),
 }
 
 
