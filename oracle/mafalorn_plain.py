@@ -74,17 +74,15 @@ def neighbour_pairs(dims: int) -> List[tuple]:
     return [(2 * i, 2 * i + 1) for i in range(dims // 2)]
 
 
-def rotate(x: torch.Tensor, pos: int, rot: dict, pairs: List[tuple]) -> torch.Tensor:
+def rotate_all(x: torch.Tensor, rot: dict, pairs: List[tuple]) -> torch.Tensor:
+    """x [T, ...]: row t turns by its position t; dimensions beyond the pairs pass unchanged."""
     out, m = x.clone(), magnitude(rot)
+    pos = torch.arange(x.shape[0], dtype=DT).reshape([-1] + [1] * (x.ndim - 2))
     for (i, j), f in zip(pairs, frequencies(rot)):
-        c, s = math.cos(pos * f) * m, math.sin(pos * f) * m
+        c, s = (torch.cos(pos * f) * m).to(x.dtype), (torch.sin(pos * f) * m).to(x.dtype)
         out[..., i] = x[..., i] * c - x[..., j] * s
         out[..., j] = x[..., j] * c + x[..., i] * s
     return out
-
-
-def rotate_all(x: torch.Tensor, rot: dict, pairs: List[tuple]) -> torch.Tensor:
-    return torch.stack([rotate(x[t], t, rot, pairs) for t in range(x.shape[0])])
 
 
 # ---- retention -----------------------------------------------------------------------------------------------------
@@ -108,14 +106,14 @@ def retention(h: torch.Tensor, p: Dict[str, torch.Tensor], c: dict, eps: float) 
 
 
 # ---- attention whose values are its unrotated keys -------------------------------------------------------------------
-def causal(i: int, j: int, size: Optional[int] = None) -> bool:
-    return j <= i and (size is None or i - j < size)
+def causal(i, j, size: Optional[int] = None):
+    """Whether position i sees position j (numbers or tensors)."""
+    return j <= i if size is None else (j <= i) & (i - j < size)
 
 
 def softmax_seen(s: torch.Tensor, size: Optional[int] = None) -> torch.Tensor:
-    T = s.shape[0]
-    seen = torch.tensor([[causal(i, j, size) for j in range(T)] for i in range(T)])
-    s = torch.where(seen, s, torch.tensor(-math.inf, dtype=s.dtype))
+    at = torch.arange(s.shape[0])
+    s = torch.where(causal(at[:, None], at[None, :], size), s, torch.tensor(-math.inf, dtype=s.dtype))
     e = torch.exp(s - s.max(-1, keepdim=True).values)
     return e / e.sum(-1, keepdim=True)
 

@@ -128,3 +128,119 @@ def run(config, tokens, dtype="float32", cuts=None, seed=0, weights=None, **kw):
     finally:
         hz.close()
     return got, oracle_logits(config, w, tokens)
+
+
+# ---- one-layer models in which token 61 asks for token 60 ------------------------------------------------------------------------
+# The stream's first quarter is a token's key address, the second quarter its query address, the second half its content.
+# Only token 60 has a key address; token 61's query address is token 60's key address.  Everything that is not needed to
+# find the marked token is zero, so its content decides the answer wherever it may be seen, and changes nothing elsewhere.
+def _addresses(w, width, g):
+    q4, half = width // 4, width // 2
+    e = w["embed"].float()
+    e[:, :half] = 0.0
+    e[60, :q4] = torch.randn(q4, generator=g)
+    e[61, q4:half] = e[60, :q4]
+    e[60, half:] *= 3.0
+    w["embed"] = e.to(torch.bfloat16)
+    w["l0.norm1"] = torch.ones(width)
+    return q4, half
+
+
+def _set(w, name, t):
+    w["l0.mix." + name] = t.to(torch.bfloat16).float()
+
+
+def latent_needle(heads=2, dim=32, vdim=16, rank=48, rot_dim=8, size=24, width=64, scale=0.4):
+    """The latent's first third holds the address, the rest the content; the rotated part is out of the way (zero)."""
+    cfg = model_config([lat(heads=heads, dim=dim, vdim=vdim, rank=rank, rot_dim=rot_dim, size=size, scale=scale, mlp=None)], width=width, vocab=64)
+    w = plain.random_weights(cfg, 33)
+    g = torch.Generator().manual_seed(34)
+    q4, half = _addresses(w, width, g)
+    third = rank // 3
+    m = torch.randn(third, q4, generator=g) * 2.0
+    dkv = torch.zeros(rank + rot_dim, width)
+    dkv[:third, :q4] = m
+    dkv[third:rank, half:] = torch.randn(rank - third, half, generator=g) / half ** 0.5
+    uk = torch.zeros(heads * dim, rank)
+    uk[:, :third] = torch.randn(heads * dim, third, generator=g) / third ** 0.5
+    uv = torch.zeros(heads * vdim, rank)
+    uv[:, third:] = torch.randn(heads * vdim, rank - third, generator=g) / rank ** 0.5
+    wq = torch.zeros(heads * (dim + rot_dim), width)
+    for h in range(heads):
+        wq[h * (dim + rot_dim):h * (dim + rot_dim) + dim, q4:half] = uk[h * dim:(h + 1) * dim, :third] @ m
+    for k, v in {"q": wq, "dkv": dkv, "dkv.norm": torch.ones(rank), "uk": uk, "uv": uv}.items():
+        _set(w, k, v)
+    return cfg, w
+
+
+def key_value_needle(heads=2, kv_heads=1, dim=32, rot_dims=8, width=64, scale=1.5):
+    """The key's rotated dimensions are zero, half of the others hold the address, the rest content that no query reads; the
+    right-hand mixer's output is zero."""
+    cfg = model_config([par(heads=heads, kv_heads=kv_heads, dim=dim, dims=rot_dims, scale=scale, left_scale=1.0, mlp=None)], width=width, vocab=64)
+    w = plain.random_weights(cfg, 37)
+    g = torch.Generator().manual_seed(38)
+    q4, half = _addresses(w, width, g)
+    a = (dim - rot_dims) // 2                                    # address dimensions behind the rotated ones
+    m = torch.randn(kv_heads, a, q4, generator=g)
+    wk = torch.zeros(kv_heads, dim, width)
+    wk[:, rot_dims:rot_dims + a, :q4] = m
+    wk[:, rot_dims + a:, half:] = torch.randn(kv_heads, dim - rot_dims - a, half, generator=g) / half ** 0.5
+    wq = torch.zeros(heads, dim, width)
+    for h in range(heads):
+        wq[h, rot_dims:rot_dims + a, q4:half] = m[h // (heads // kv_heads)]
+    _set(w, "left.q", wq.reshape(-1, width))
+    _set(w, "left.k", wk.reshape(-1, width))
+    _set(w, "right.o", torch.zeros_like(w["l0.mix.right.o"].float()))
+    return cfg, w
+
+
+def retention_needle(heads=2, dim=16, vdim=24, width=64):
+    """Decays near one and nothing rotated but two dimensions that stay zero, so the one key written stays readable far away."""
+    cfg = model_config([ret(heads=heads, dim=dim, vdim=vdim, decay=[1.0 - 2.0 ** -10, 1.0][:heads], dims=2, mlp=None)], width=width, vocab=64)
+    w = plain.random_weights(cfg, 35)
+    g = torch.Generator().manual_seed(36)
+    q4, half = _addresses(w, width, g)
+    m = torch.randn(heads, dim, q4, generator=g)
+    m[:, :2] = 0.0
+    wk, wq = torch.zeros(heads * dim, width), torch.zeros(heads * dim, width)
+    wk[:, :q4] = m.reshape(-1, q4)
+    wq[:, q4:half] = m.reshape(-1, q4)
+    wv = torch.zeros(heads * vdim, width)
+    wv[:, half:] = torch.randn(heads * vdim, half, generator=g) / half ** 0.5
+    _set(w, "q", wq)
+    _set(w, "k", wk)
+    _set(w, "v", wv)
+    return cfg, w
+
+
+def delta_needle(heads=2, kv_heads=1, dim=16, vdim=24, conv=3, width=64):
+    """Decays near one, convolutions that pass the current token only; the left-hand mixer's output is zero."""
+    cfg = model_config([par(d_heads=heads, d_kv_heads=kv_heads, d_dim=dim, d_vdim=vdim, conv=conv, right_scale=1.0, mlp=None)], width=width, vocab=64)
+    w = plain.random_weights(cfg, 39)
+    g = torch.Generator().manual_seed(40)
+    q4, half = _addresses(w, width, g)
+    m = torch.randn(kv_heads * dim, q4, generator=g)
+    wk, wq = torch.zeros(kv_heads * dim, width), torch.zeros(kv_heads * dim, width)
+    wk[:, :q4] = m
+    wq[:, q4:half] = m
+    wv = torch.zeros(heads * vdim, width)
+    wv[:, half:] = torch.randn(heads * vdim, half, generator=g) / half ** 0.5
+    for name, t in (("q", wq), ("k", wk), ("v", wv)):
+        _set(w, f"right.{name}", t)
+        taps = torch.zeros(t.shape[0], conv)
+        taps[:, -1] = 1.0
+        _set(w, f"right.{name}.conv", taps)
+    _set(w, "right.A_log", torch.full((heads,), -9.0))
+    _set(w, "right.a", torch.zeros(heads, width))
+    _set(w, "right.dt_bias", torch.zeros(heads))
+    _set(w, "left.o", torch.zeros_like(w["l0.mix.left.o"].float()))
+    return cfg, w
+
+
+def needle_tokens(n, needle_at):
+    """(tokens with the marked token and the asking token last, the same without the marked token)."""
+    toks = [2 + (i % 50) for i in range(n)]
+    without = list(toks)
+    toks[needle_at] = 60
+    toks[-1] = without[-1] = 61
+    return toks, without
