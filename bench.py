@@ -587,6 +587,32 @@ def run_compare_kisadra(args):
                       "peaks": peaks, "clocks": clocks, "results": res}))
 
 
+def run_compare_mafalorn(args):
+    """Option --compare-mafalorn: Mafalorn (retention / attention beside a delta rule / windowed latent attention, experts in every
+    layer) beside the closest existing models, Kisadra and Kinetar, at equal width, layer runs, heads and active feed-forward
+    size; device times from CUDA events, three warm-up passes, weights + activations larger than L2."""
+    import __graft_entry__ as g
+    g.build()
+    from jacobiforcing_b200 import hybrid_bench as hb
+    try:
+        with open(os.path.join(ROOT, "MEASURED_PEAKS.json")) as f:
+            mp = json.load(f)
+        peaks = {"hbm_gbs": float(mp["hbm_gbs"]), "bf16_tflops": float(mp["bf16_tflops"]), "source": "measured"}
+    except Exception:
+        peaks = {"hbm_gbs": 6650.0, "bf16_tflops": 1590.0, "source": "fallback"}
+    mon = ClockSampler(0)
+    mon.start()
+    res = []
+    for size in args.compare_mafalorn.split(","):
+        row = {"size": size}
+        for design in ("Mafalorn", "Kisadra", "Kinetar"):
+            row[design.lower()] = hb.run_hybrid(size, args.hybrid_prompt, args.hybrid_decode_steps, [1, 8], peaks, design=design)
+        res.append(row)
+    clocks = mon.stop()
+    print(json.dumps({"metric": "mafalorn_vs_kisadra_and_kinetar_throughput", "unit": "tokens/s", "dtype": "bf16", "data": "synthetic",
+                      "peaks": peaks, "clocks": clocks, "results": res}))
+
+
 def main():
     ap = argparse.ArgumentParser()
     ap.add_argument("--gpus", type=int, default=1)
@@ -626,6 +652,9 @@ def main():
     ap.add_argument("--compare-kisadra", default="", metavar="SIZES",
                     help="instead of the headline workload: prefill / decode throughput of Kisadra beside Famepel and Sebavik at "
                          "equal size, e.g. w1024,w2048 (one JSON line)")
+    ap.add_argument("--compare-mafalorn", default="", metavar="SIZES",
+                    help="instead of the headline workload: prefill / decode throughput of Mafalorn beside Kisadra and Kinetar at "
+                         "equal size, e.g. w1024,w2048 (one JSON line)")
     ap.add_argument("--hybrid-prompt", type=int, default=4096)
     ap.add_argument("--hybrid-decode-steps", type=int, default=35)
     args = ap.parse_args()
@@ -643,6 +672,9 @@ def main():
         return
     if args.compare_kisadra:
         run_compare_kisadra(args)
+        return
+    if args.compare_mafalorn:
+        run_compare_mafalorn(args)
         return
     if args.warmup < 3 and args.impl == "ours":
         args.warmup = 3                                  # timing rule: at least three warm-up steps

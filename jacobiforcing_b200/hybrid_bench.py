@@ -8,7 +8,10 @@ attention and routed experts).  `bench.py --compare-sebavik`: Sebavik beside Vos
 attention over paged keys and values, a gated dense feed-forward alternating with routed experts, RMS norms).  `bench.py
 --compare-kisadra`: Kisadra beside Famepel at equal width / layer runs / active feed-forward size (both: a matrix-state
 recurrence in heads of 128 x 128, latent attention over the same rank, routed gated experts) and beside Sebavik, whose
-attention with a distance bias is the like kernel of the chunk attention."""
+attention with a distance bias is the like kernel of the chunk attention.  `bench.py --compare-mafalorn`: Mafalorn beside Kisadra at
+equal width / layer runs / active feed-forward size (both: a matrix-state recurrence in heads of 128 x 128, latent attention over
+the same rank, gated experts beside identity experts) and beside Kinetar, whose delta rule and attention valued by its keys
+are the like kernels of the "parallel" mixer."""
 from __future__ import annotations
 
 import time
@@ -308,6 +311,96 @@ def kisadra_weights(desc: dict, seed: int, low: int = 16) -> Dict[str, np.ndarra
     return w
 
 
+def mafalorn_description(sz: dict) -> dict:
+    """Layers in the order retention, attention beside delta rule, retention, latent attention.  Retention and delta rule in heads of
+    128 keys x 128 values (values = width), attention in heads of 128 with half of each head rotated (interpolated from 4096
+    positions), latent attention with a rank of 512 + 64 rotated inside a window of 1024; experts of ff / top each (8 x top of them
+    and `top` identity experts, `top` per token from half of the groups) in every layer."""
+    W, top = sz["width"], sz.get("top", 4)
+    n = W // 128
+    moe = {"kind": "moe", "expert": {"ff": sz["ff"] // top},
+           "router": {"experts": 8 * top, "top": top, "identity": top, "groups": {"count": 4, "keep": 2}}}
+    ret = {"type": "retention", "mixer": {"heads": n, "dim": 128, "vdim": 128, "decay": [1.0 - 2.0 ** (-5.0 - 4.0 * h / n) for h in range(n)],
+                                          "rot": {"base": 10000.0, "dims": 128}}, "mlp": moe}
+    par = {"type": "parallel",
+           "mixer": {"left": {"heads": sz["heads"], "kv_heads": sz["kv_heads"], "dim": sz["dim"], "vdim": sz["dim"], "scale": sz["dim"] ** -0.5,
+                              "rot": {"base": 10000.0, "dims": sz["dim"] // 2,
+                                      "scaling": {"factor": 4.0, "original": 4096, "fast": 32.0, "slow": 1.0}}}, "left_scale": 0.7,
+                     "right": {"heads": n, "kv_heads": max(1, n // 2), "dim": 128, "vdim": 128, "conv": 4}, "right_scale": 0.7}, "mlp": moe}
+    lat = {"type": "latent_attention", "mixer": {"heads": sz["heads"], "dim": 128, "rot_dim": 64, "vdim": 128, "kv_rank": sz.get("kv_rank", 512),
+                                                 "scale": 192 ** -0.5, "rot": {"base": 10000.0, "dims": 64}, "mask": {"size": 1024}}, "mlp": moe}
+    return {"architecture": "Mafalorn", "layers": [[ret, par, ret, lat][i % 4] for i in range(sz["layers"])], "logit_scale": 1.0,
+            "norm": {"eps": 1e-6}, "vocab": sz["vocab"], "width": W}
+
+
+def mafalorn_weights(desc: dict, seed: int) -> Dict[str, np.ndarray]:
+    rng = np.random.default_rng(seed)
+    W, V = desc["width"], desc["vocab"]
+
+    def lin(n, k):
+        return (rng.standard_normal((n, k), dtype=np.float32) / np.sqrt(k)).astype(np.float32)
+
+    def vec(n, s=0.1, b=0.0):
+        return (rng.standard_normal(n, dtype=np.float32) * s + b).astype(np.float32)
+    w = {"embed": lin(V, W) * 4.0, "final.norm": vec(W, 0.1, 1.0), "head": lin(V, W)}
+    for i, lc in enumerate(desc["layers"]):
+        p, m, M = f"l{i}.", lc["mixer"], f"l{i}.mix."
+        for n in ("norm1", "norm1b", "norm2", "norm2b"):
+            w[p + n] = vec(W, 0.1, 1.0)
+        if lc["type"] == "retention":
+            nq, nv = m["heads"] * m["dim"], m["heads"] * m["vdim"]
+            w.update({M + "q": lin(nq, W), M + "k": lin(nq, W), M + "v": lin(nv, W), M + "g": lin(nv, W), M + "o": lin(W, nv)})
+        elif lc["type"] == "parallel":
+            a, d = m["left"], m["right"]
+            L, R = M + "left.", M + "right."
+            nq, H, nk, nv = a["heads"] * a["dim"], d["heads"], d["kv_heads"] * d["dim"], d["heads"] * d["vdim"]
+            w.update({L + "q": lin(nq, W), L + "k": lin(a["kv_heads"] * a["dim"], W), L + "g": lin(a["heads"], W), L + "o": lin(W, nq),
+                      R + "q": lin(nk, W), R + "k": lin(nk, W), R + "v": lin(nv, W), R + "q.conv": vec((nk, d["conv"]), 0.5),
+                      R + "k.conv": vec((nk, d["conv"]), 0.5), R + "v.conv": vec((nv, d["conv"]), 0.5), R + "b": lin(H, W), R + "a": lin(H, W),
+                      R + "A_log": np.log(rng.uniform(0.1, 1.5, H)).astype(np.float32), R + "dt_bias": vec(H, 0.5, -1.0),
+                      R + "norm": vec(d["vdim"], 0.2, 1.0), R + "g": lin(nv, W), R + "o": lin(W, nv)})
+        else:
+            H, K, r = m["heads"], m["kv_rank"], m["rot_dim"]
+            nv = H * m["vdim"]
+            w.update({M + "q": lin(H * (m["dim"] + r), W), M + "dkv": lin(K + r, W), M + "dkv.norm": vec(K, 0.1, 1.0), M + "uk": lin(H * m["dim"], K),
+                      M + "uv": lin(nv, K), M + "g": lin(nv, W), M + "o": lin(W, nv)})
+        mlp = lc["mlp"]
+        ff, E, n = mlp["expert"]["ff"], mlp["router"]["experts"], mlp["router"]["experts"] + mlp["router"]["identity"]
+        w[p + "mlp.router"], w[p + "mlp.correction"] = lin(n, W) * 2.0, vec(n, 0.01)
+        for e in range(E):
+            w[f"{p}mlp.e{e}.gate"], w[f"{p}mlp.e{e}.up"], w[f"{p}mlp.e{e}.down"] = lin(ff, W), lin(ff, W), lin(W, ff)
+    return w
+
+
+def _mafalorn_costs(desc: dict, hc, prompt: int) -> dict:
+    """Multiply-adds per token per kernel group; experts as if no choice were an identity expert."""
+    W = desc["width"]
+    per = {"gemm_in": 0, "gemm_out": 0, "small_gemm": 0, "experts": 0, "expert_weights": 0, "delta": 0, "attention_prompt": 0}
+    for s in hc.layers:
+        if s.mixer == 9:
+            nq, nv = s.g_heads * s.g_dim, s.g_heads * s.g_vdim
+            per["gemm_in"] += (2 * nq + 2 * nv) * W
+            per["gemm_out"] += nv * W
+            per["delta"] += 2 * nq * s.g_vdim
+        elif s.mixer == 10:
+            nq, nk, nv = s.b_heads * s.b_dim, s.b_kv_heads * s.b_dim, s.d_heads * s.d_vdim
+            per["gemm_in"] += (nq + nk + s.b_heads + 2 * s.d_kv_heads * s.d_dim + 2 * nv + 2 * s.d_heads) * W
+            per["gemm_out"] += (nq + nv) * W
+            per["delta"] += 3 * s.d_heads * s.d_dim * s.d_vdim
+            per["attention_prompt"] += prompt * (prompt + 1) // 2 * nq * 2
+        else:
+            per["gemm_in"] += (s.l_heads * (s.l_dim + s.l_rot_dim + s.l_vdim) + s.l_kv_rank + s.l_rot_dim) * W
+            per["gemm_out"] += s.l_heads * s.l_vdim * W
+            per["small_gemm"] += s.l_heads * (s.l_dim + s.l_vdim) * s.l_kv_rank
+            seen = sum(min(i + 1, s.l_window or prompt) for i in range(prompt))
+            per["attention_prompt"] += seen * s.l_heads * (2 * s.l_kv_rank + s.l_rot_dim)
+        if s.ff_kind == 2:
+            per["experts"] += s.x_top * 3 * s.ff * W
+            per["expert_weights"] += s.x_experts * 3 * s.ff * W
+    per["head"] = desc["vocab"] * W
+    return per
+
+
 def _kisadra_costs(desc: dict, hc, prompt: int) -> dict:
     """Multiply-adds per token per kernel group (gate / up, router and the loop projection run inside or beside the input
     product, the dense down-projection inside the output product); experts as if no choice were an identity expert."""
@@ -425,6 +518,8 @@ def _hybrid_costs(desc: dict, hc, prompt: int = 0) -> dict:
         return _sebavik_costs(desc, hc, prompt)
     if desc["architecture"] == "Kisadra":
         return _kisadra_costs(desc, hc, prompt)
+    if desc["architecture"] == "Mafalorn":
+        return _mafalorn_costs(desc, hc, prompt)
     W = desc["width"]
     per = {"gemm_in": 0, "gemm_out": 0, "small_gemm": 0}
     for s in hc.layers:
@@ -461,6 +556,9 @@ def run_hybrid(size: str, prompt: int, decode_steps: int, batches: List[int], pe
     elif design == "Kisadra":
         desc = kisadra_description(sz)
         w = kisadra_weights(desc, seed)
+    elif design == "Mafalorn":
+        desc = mafalorn_description(sz)
+        w = mafalorn_weights(desc, seed)
     else:
         desc = hybrid_description(sz)
         w = hybrid_weights(desc, seed)

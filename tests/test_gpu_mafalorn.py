@@ -176,7 +176,7 @@ def test_constant_matters_and_is_honoured(what):
     elif what == "keep":
         cfg2["layers"][1]["mlp"]["router"]["groups"]["keep"] = 1
     elif what in ("factor", "original", "fast", "slow"):
-        m[1]["left"]["rot"]["scaling"][what] *= {"factor": 1.3, "original": 2, "fast": 0.4, "slow": 3.0}[what]
+        m[1]["left"]["rot"]["scaling"][what] *= {"factor": 1.3, "original": 2, "fast": 0.1, "slow": 3.0}[what]
     elif what in ("head norm", "latent norm", "norm behind the mixer", "norm behind the experts", "decay bias", "A_log"):
         name = {"head norm": "l1.mix.right.norm", "latent norm": "l2.mix.dkv.norm", "norm behind the mixer": "l1.norm1b",
                 "norm behind the experts": "l0.norm2b", "decay bias": "l1.mix.right.dt_bias", "A_log": "l1.mix.right.A_log"}[what]
@@ -431,7 +431,7 @@ def test_other_sizes(idx, dtype):
 # layer-sized models (the tensor-core products, attention tiles and sorted experts take over in the bf16 build): unlike head
 # shapes, windows over several 64-token pages and inside one, feed-forwards beside every mixer
 LAYER_SIZED = [
-    model_config([lat(heads=4, dim=48, rot_dim=32, vdim=40, rank=96, scale=0.11, base=10000.0, size=100, mlp=moe(10, 2, 96, 2, (3, 2))),
+    model_config([lat(heads=4, dim=48, rot_dim=32, vdim=40, rank=96, scale=0.11, base=10000.0, size=100, mlp=moe(10, 2, 96, 2, (4, 2))),
                   ret(heads=5, dim=48, vdim=64, base=10000.0, mlp=moe(8, 2, 96, 4, (2, 1))),
                   par(heads=8, kv_heads=2, dim=40, dims=24, scale=0.16, base=10000.0, d_heads=6, d_kv_heads=3, d_dim=48, d_vdim=64, conv=4,
                       mlp=moe(9, 3, 64, 0, (3, 2))),
@@ -441,7 +441,6 @@ LAYER_SIZED = [
                   ret(heads=3, dim=24, vdim=88, mlp=moe(7, 3, 50, 2, (3, 2))),
                   lat(heads=6, dim=40, rot_dim=24, vdim=40, rank=40, scale=0.12, base=5000.0, size=257, mlp=moe(6, 2, 72, 0, None))], width=200, vocab=333),
 ]
-LAYER_SIZED[0]["layers"][0]["mlp"]["router"]["groups"] = {"count": 4, "keep": 2}
 
 
 @pytest.mark.parametrize("idx", range(len(LAYER_SIZED)))
