@@ -77,47 +77,22 @@ def row_errs(got: np.ndarray, want: np.ndarray) -> np.ndarray:
     return np.sqrt((d ** 2).mean(1)) / np.sqrt((w ** 2).mean(1) + 1e-30)
 
 
-TOL = {"float32": 2e-4, "bfloat16": 6e-2}
+TOL = {"float32": 2e-4, "bfloat16": 8e-2}
 
 
-def close(got, want, dtype="float32", skip=()) -> bool:
-    """float32: every row within the tolerance.  bfloat16: the rows in `skip` are not judged (see near_ties); of the others a
-    fifth may lie outside (typical rows are several times below the tolerance)."""
+def close(got, want, dtype="float32") -> bool:
+    """float32: every row within the tolerance.  bfloat16: one row in twenty (at least one) may lie outside, up to four times: a
+    sublayer whose result happens to be small is normed up, rounding and all.  Runs of models with routers use `settled`
+    weights there: rounding may choose another expert at a near tie, and every later row sees it through states and keys."""
     e = row_errs(got, want)
     if dtype == "float32":
         return bool(e.max() < TOL[dtype])
-    keep = np.ones(len(e), dtype=bool)
-    keep[[i for i in skip if i < len(e)]] = False
-    if not keep.any():
-        return True
-    e = e[keep]
-    return bool(np.mean(e < TOL[dtype]) >= 0.8 and np.median(e) < TOL[dtype] / 2)
+    return bool(np.sum(e >= TOL[dtype]) <= max(1, 0.05 * len(e)) and e.max() < 4 * TOL[dtype] and np.median(e) < TOL[dtype] / 1.5)
 
 
-def near_ties(config, weights, tokens, margin=0.01):
-    """Rows where the last chosen and the first rejected output, or the last kept and the first dropped group, lie closer than
-    `margin` in the oracle: a run with rounding may choose the other one."""
-    found = []
-    inner = plain.route
-
-    def watching(h, router, correction, r):
-        choice = torch.softmax(h @ router.T, 1) + correction
-        n, gr = choice.shape[1], r.get("groups") or {"count": 1, "keep": 1}
-        worth = choice.reshape(-1, gr["count"], n // gr["count"]).max(2).values
-        z, keep = torch.sort(worth, 1, descending=True)
-        if gr["keep"] < gr["count"]:
-            found.extend(torch.nonzero(z[:, gr["keep"] - 1] - z[:, gr["keep"]] < margin).flatten().tolist())
-        for t in range(choice.shape[0]):
-            c = torch.sort(choice[t].reshape(gr["count"], -1)[keep[t, :gr["keep"]]].flatten(), descending=True).values
-            if r["top"] < len(c) and c[r["top"] - 1] - c[r["top"]] < margin:
-                found.append(t)
-        return inner(h, router, correction, r)
-    plain.route = watching
-    try:
-        plain.forward(config, weights, list(tokens))
-    finally:
-        plain.route = inner
-    return sorted(set(found))
+def settled(weights):
+    """The same weights with corrections so large that they alone decide the choice of experts: no rounding can flip it."""
+    return {k: (v.float() * 1000.0 if k.endswith(".correction") else v) for k, v in weights.items()}
 
 
 def run(config, tokens, dtype="float32", cuts=None, seed=0, weights=None, **kw):
