@@ -401,6 +401,37 @@ constexpr size_t attn_wide_smem(int dk) {
   return (size_t)2 * 64 * (((dk + 15) & ~15) + 8) * 2 + (size_t)2 * 64 * 72 * 2 + (256 + 192) * 4;
 }
 
+// Weights of a row's n key splits (maximum, denominator per split in ml) merged with a sink logit (-inf: none), times scale:
+// made by the first warp, in shared memory for the whole block on return.
+constexpr int HY_MAX_SPLITS = 272;
+__device__ __forceinline__ void split_weights(const float* __restrict__ ml, int n, float sink, float scale, float* wt) {
+  if (threadIdx.x < 32) {
+    float M = -INFINITY;
+    for (int s = threadIdx.x; s < n; s += 32) M = fmaxf(M, ml[2 * s]);
+    M = fmaxf(warp_max(M), sink);
+    float L = 0.0f;
+    for (int s = threadIdx.x; s < n; s += 32) {
+      const float e = expf(ml[2 * s] - M);
+      wt[s] = e;
+      L = fmaf(ml[2 * s + 1], e, L);
+    }
+    const float f = scale / (warp_sum(L) + expf(sink - M));
+    for (int s = threadIdx.x; s < n; s += 32) wt[s] *= f;
+  }
+  __syncthreads();
+}
+// four values of a row over its splits (rows `stride` floats apart, 16-byte aligned)
+__device__ __forceinline__ float4 merge_splits(const float* __restrict__ po, int stride, int n, const float* wt) {
+  float4 a = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+#pragma unroll 4
+  for (int s = 0; s < n; ++s) {
+    const float4 v = *reinterpret_cast<const float4*>(po + (size_t)s * stride);
+    const float w = wt[s];
+    a.x = fmaf(v.x, w, a.x); a.y = fmaf(v.y, w, a.y); a.z = fmaf(v.z, w, a.z); a.w = fmaf(v.w, w, a.w);
+  }
+  return a;
+}
+
 // Merge the key splits of one (token, head) with the sink, gate the result, scale it, write the projection's operand.
 // part_o rows are dim wide; the first vdim of them are values.  G: key heads (a row's tile is found from it).
 template <typename WT, typename OT>
@@ -417,17 +448,28 @@ __global__ void attn_combine_kernel(Batch b, const float* __restrict__ part_o, c
     live -= tile;
   }
   const float sk = sink ? to_f(sink[h]) : -INFINITY;       // sink NULL: an ordinary softmax
-  const size_t slot0 = ((size_t)t * H + h) * n_splits;
-  float M = sk;
-  for (int s = from; s < live; ++s) M = fmaxf(M, part_ml[(slot0 + s) * 2]);
-  float L = expf(sk - M);
-  for (int s = from; s < live; ++s) L += part_ml[(slot0 + s) * 2 + 1] * expf(part_ml[(slot0 + s) * 2] - M);
-  const float inv = 1.0f / L;
+  const size_t slot0 = ((size_t)t * H + h) * n_splits + from;
+  const int n = live - from;
+  __shared__ float wt[HY_MAX_SPLITS];
+  split_weights(part_ml + slot0 * 2, n, sk, out_scale, wt);
+  const float* po = part_o + slot0 * dim;
+  if (vdim % 4 == 0) {
+    for (int d = threadIdx.x * 4; d < vdim; d += blockDim.x * 4) {
+      const float4 a = merge_splits(po + d, dim, n, wt);
+      const float v[4] = {a.x, a.y, a.z, a.w};
+#pragma unroll
+      for (int j = 0; j < 4; ++j) {
+        const float gt = gate ? sigmoid_f(to_f(gate[(size_t)t * ldg + h * vdim + d + j])) : 1.0f;
+        out[(size_t)t * ldo + h * vdim + d + j] = from_f<OT>(v[j] * gt);
+      }
+    }
+    return;
+  }
   for (int d = threadIdx.x; d < vdim; d += blockDim.x) {
     float acc = 0.0f;
-    for (int s = from; s < live; ++s) acc += part_o[(slot0 + s) * dim + d] * expf(part_ml[(slot0 + s) * 2] - M);
+    for (int s = 0; s < n; ++s) acc = fmaf(po[(size_t)s * dim + d], wt[s], acc);
     const float gt = gate ? sigmoid_f(to_f(gate[(size_t)t * ldg + h * vdim + d])) : 1.0f;
-    out[(size_t)t * ldo + h * vdim + d] = from_f<OT>(acc * inv * gt * out_scale);
+    out[(size_t)t * ldo + h * vdim + d] = from_f<OT>(acc * gt);
   }
 }
 

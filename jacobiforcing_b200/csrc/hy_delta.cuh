@@ -141,7 +141,13 @@ __global__ void __launch_bounds__(128) delta_head_kernel(Batch b, const AT* __re
     if (ahead) jf::cp_async_wait_all();
     __syncthreads();                                           // raw rows have landed; the previous batch is finished
     const AT* src = raw + (size_t)buf * TB * RW;
-    // unit vectors and the token's scalars: one warp per token
+    // decays and step sizes: one thread per token; unit vectors and k.q: one warp per token
+    float* scf = reinterpret_cast<float*>(sc);
+    if (tid < nb) {
+      const size_t t = (size_t)(start + j0 + tid);
+      scf[4 * tid] = expf(-rate * softplus_f(ba[t * ldba + H + h] + bias));
+      scf[4 * tid + 1] = sigmoid_f(ba[t * ldba + h]);
+    }
     for (int tt = warp; tt < nb; tt += 4) {
       constexpr int EL = (DR + 31) / 32;
       const size_t t = (size_t)(start + j0 + tt);
@@ -162,8 +168,7 @@ __global__ void __launch_bounds__(128) delta_head_kernel(Batch b, const AT* __re
         const int k = lane + 32 * i;
         if (k < DR) { sq[tt * DR + k] = qv[i] * qi; sk[tt * DR + k] = kv[i] * ki; }
       }
-      if (lane == 0)
-        sc[tt] = make_float4(expf(-rate * softplus_f(ba[t * ldba + H + h] + bias)), sigmoid_f(ba[t * ldba + h]), qk * qi * ki, 0.0f);
+      if (lane == 0) scf[4 * tt + 2] = qk * qi * ki;
     }
     for (int i = tid; i < nb * CPB; i += 128) {
       const int tt = i / CPB, k = i % CPB;

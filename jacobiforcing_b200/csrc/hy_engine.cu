@@ -1502,12 +1502,16 @@ const UnitList* attn_units(hy_engine* h, int E, int T, int H, int G, bool any_ra
   int maxctx = 1;
   for (int e = 0; e < E; ++e) maxctx = std::max(maxctx, h->step_pos0[e] + h->step_start[e + 1] - h->step_start[e]);
   const int ns_cap = (int)std::max<size_t>(1, h->part_rows / ((size_t)T * H));
-  int ns = std::min(std::min((maxctx + 255) / 256, ns_cap), 256);
+  // key splits of 256 keys; shorter ones (down to a tile of 64) while a step of few rows leaves SMs without a unit
+  size_t tiles = 0;
+  for (int e = 0; e < E; ++e) tiles += (size_t)G * ((size_t)(h->step_start[e + 1] - h->step_start[e]) * R / 64 + 1);
+  auto splits_of = [&](int keys) { return std::max((keys + 255) / 256, std::min((keys + 63) / 64, (int)(148 / tiles))); };
+  int ns = std::min(std::min(splits_of(maxctx), ns_cap), 256);
   int split = ((maxctx + ns - 1) / ns + 63) / 64 * 64;
   ns = (maxctx + split - 1) / split;
   const int seen = window > 0 ? window + 63 / R : maxctx;     // most keys a tile of 64 rows sees
   if (seen < maxctx && ns_cap >= 2) {
-    const int n = std::min(std::min((seen + 255) / 256, ns_cap - 1), 255);
+    const int n = std::min(std::min(splits_of(seen), ns_cap - 1), 255);
     split = ((seen + n - 1) / n + 63) / 64 * 64;
     ns = std::min((seen + split - 1) / split + 1, (maxctx + split - 1) / split);
   } else if (seen < maxctx) {
@@ -1642,7 +1646,7 @@ void latent_mixer(hy_engine* h, const Batch& b, const LayerW& L, const hy_layer_
         else if (nt == 4) attn_wide_kernel<4><<<u->n, 256, smem, s>>>(HY_WIDE_ARGS);
         else attn_wide_kernel<8><<<u->n, 256, smem, s>>>(HY_WIDE_ARGS);
 #undef HY_WIDE_ARGS
-        attn_combine_kernel<WT, float><<<T * H, 64, 0, s>>>(b, h->part_o, h->part_ml, (const WT*)L.sink, nullptr, 0, H, 1, pstride, R,
+        attn_combine_kernel<WT, float><<<T * H, 128, 0, s>>>(b, h->part_o, h->part_ml, (const WT*)L.sink, nullptr, 0, H, 1, pstride, R,
                                                             c.l_window, u->split, u->ns, 1.0f, h->f2, h->ld_f2);
         h->launches += 2;
       }
@@ -2192,16 +2196,16 @@ void biased_attend(hy_engine* h, const Batch& b, const LayerW& L, const hy_layer
         tc = true;
         static bool attr = false;
         if (!attr) {
-          cudaFuncSetAttribute(biased_mma_kernel<64>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)window_mma_smem(64));
-          cudaFuncSetAttribute(biased_mma_kernel<128>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)window_mma_smem(128));
+          cudaFuncSetAttribute(biased_mma_kernel<64, 2>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)window_mma_smem(64));
+          cudaFuncSetAttribute(biased_mma_kernel<128, 1>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)window_mma_smem(128) / 2);
+          cudaFuncSetAttribute(biased_mma_kernel<128, 2>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)window_mma_smem(128));
           attr = true;
         }
-        if (dp == 64)
-          biased_mma_kernel<64><<<u->n, 128, window_mma_smem(64), s>>>(b, u->d, pin + L.c_q, h->ld_pin, bc, (const bf16*)L.cache,
-                                                                            (const bf16*)L.cache_v, cat, h->ld_cat, u->ns, h->part_o, h->part_ml);
-        else
-          biased_mma_kernel<128><<<u->n, 128, window_mma_smem(128), s>>>(b, u->d, pin + L.c_q, h->ld_pin, bc, (const bf16*)L.cache,
-                                                                              (const bf16*)L.cache_v, cat, h->ld_cat, u->ns, h->part_o, h->part_ml);
+#define HY_BIASED_ARGS b, u->d, pin + L.c_q, h->ld_pin, bc, (const bf16*)L.cache, (const bf16*)L.cache_v, cat, h->ld_cat, u->ns, h->part_o, h->part_ml
+        if (dp == 64) biased_mma_kernel<64, 2><<<u->n, 128, window_mma_smem(64), s>>>(HY_BIASED_ARGS);
+        else if (u->n > 148) biased_mma_kernel<128, 1><<<u->n, 128, window_mma_smem(128) / 2, s>>>(HY_BIASED_ARGS);
+        else biased_mma_kernel<128, 2><<<u->n, 128, window_mma_smem(128), s>>>(HY_BIASED_ARGS);
+#undef HY_BIASED_ARGS
         if (u->ns > 1) {
           biased_combine_kernel<bf16><<<T * c.b_heads, 64, 0, s>>>(h->part_o, h->part_ml, bc, dp, u->ns, cat, h->ld_cat);
           h->launches++;
@@ -2413,11 +2417,16 @@ void launch_row_close(hy_engine* h, int T, RowClose rc) {
   typedef AT WT;
   const int W = h->m.width;
   static bool attr = false;                                  // per AT: this function is a template
-  if (!attr) { cudaFuncSetAttribute(row_close_kernel<AT, WT>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024); attr = true; }
+  if (!attr) {
+    cudaFuncSetAttribute(row_close_kernel<AT, WT, 1>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
+    cudaFuncSetAttribute(row_close_kernel<AT, WT, 4>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
+    attr = true;
+  }
   rc.eps = h->m.norm_eps;
   if (!rc.rows && !rc.y && !rc.cast_out && !rc.norm_w) return;
   ProfScope ps(h, HY_PROF_NORM);
-  row_close_kernel<AT, WT><<<T, 256, (size_t)W * 4, h->stream>>>(rc, W, h->x, (AT*)h->hbuf);
+  if (W % 4 == 0) row_close_kernel<AT, WT, 4><<<T, 256, (size_t)W * 4, h->stream>>>(rc, W, h->x, (AT*)h->hbuf);
+  else row_close_kernel<AT, WT, 1><<<T, 256, (size_t)W * 4, h->stream>>>(rc, W, h->x, (AT*)h->hbuf);
   h->launches++;
 }
 

@@ -273,46 +273,93 @@ struct RowClose {
   const float* y; int ldy; const void* post_w;
 };
 
-template <typename AT, typename WT>
+// V channels per thread at a time (V = 4: width and all leading dimensions are multiples of 4).
+constexpr int HY_CLOSE_TOP = 64;                               // choices whose rows and weights are staged in shared memory
+template <typename AT, typename WT, int V>
 __global__ void __launch_bounds__(256) row_close_kernel(RowClose c, int width, float* __restrict__ x, AT* h) {
+  typedef VecN<float, V> F;
   extern __shared__ __align__(16) unsigned char hy_smem[];
   float* xs = reinterpret_cast<float*>(hy_smem);               // [width]
   __shared__ float red[33];
+  __shared__ int srow[HY_CLOSE_TOP];
+  __shared__ float swt[HY_CLOSE_TOP];
   const int t = blockIdx.x;
+  const int first = threadIdx.x * V, step = blockDim.x * V;
+  const bool adds = c.rows || c.y;
+  if (c.rows) {                                                // row of every staged choice, -1: an identity choice
+    for (int k = threadIdx.x; k < min(c.top, HY_CLOSE_TOP); k += blockDim.x) {
+      const int i = t * c.top + k;
+      srow[k] = c.ids[i] >= c.n_experts ? -1 : c.pair_row ? c.pair_row[i] : i;
+      swt[k] = c.wts[i];
+    }
+    __syncthreads();
+  }
   float ss = 0.0f;
   auto result = [&](int ch) {
-    if (c.y) return c.y[(size_t)t * c.ldy + ch];
-    float y = 0.0f;
+    if (c.y) return *reinterpret_cast<const F*>(c.y + (size_t)t * c.ldy + ch);
+    F y{}, own{};
+    {
+      const VecN<AT, V> hv = *reinterpret_cast<const VecN<AT, V>*>(h + (size_t)t * width + ch);
+#pragma unroll
+      for (int j = 0; j < V; ++j) own.v[j] = to_f(hv.v[j]);
+    }
+#pragma unroll 4
     for (int k = 0; k < c.top; ++k) {
-      const int i = t * c.top + k;
-      const float r = c.ids[i] >= c.n_experts ? to_f(h[(size_t)t * width + ch])
-                                              : c.rows[(size_t)(c.pair_row ? c.pair_row[i] : i) * c.ldr + ch];
-      y = fmaf(c.wts[i], r, y);
+      int row; float w;
+      if (k < HY_CLOSE_TOP) { row = srow[k]; w = swt[k]; }
+      else {
+        const int i = t * c.top + k;
+        row = c.ids[i] >= c.n_experts ? -1 : c.pair_row ? c.pair_row[i] : i;
+        w = c.wts[i];
+      }
+      const F r = row < 0 ? own : *reinterpret_cast<const F*>(c.rows + (size_t)row * c.ldr + ch);
+#pragma unroll
+      for (int j = 0; j < V; ++j) y.v[j] = fmaf(w, r.v[j], y.v[j]);
     }
     return y;
   };
   float pinv = 1.0f;
   if (c.post_w) {
-    for (int ch = threadIdx.x; ch < width; ch += blockDim.x) { const float y = result(ch); xs[ch] = y; ss = fmaf(y, y, ss); }
+    for (int ch = first; ch < width; ch += step) {
+      const F y = result(ch);
+      *reinterpret_cast<F*>(xs + ch) = y;
+#pragma unroll
+      for (int j = 0; j < V; ++j) ss = fmaf(y.v[j], y.v[j], ss);
+    }
     pinv = 1.0f / sqrtf(block_sum(ss, red) / (float)width + c.eps);
     ss = 0.0f;
   }
-  for (int ch = threadIdx.x; ch < width; ch += blockDim.x) {
-    float v = x[(size_t)t * width + ch];
-    if (c.rows || c.y) {
-      v += c.post_w ? xs[ch] * pinv * to_f(((const WT*)c.post_w)[ch]) : result(ch);
-      x[(size_t)t * width + ch] = v;
+  for (int ch = first; ch < width; ch += step) {
+    F v = *reinterpret_cast<const F*>(x + (size_t)t * width + ch);
+    if (adds) {
+      if (c.post_w) {
+        const F y = *reinterpret_cast<const F*>(xs + ch);
+        const VecN<WT, V> w = *reinterpret_cast<const VecN<WT, V>*>((const WT*)c.post_w + ch);
+#pragma unroll
+        for (int j = 0; j < V; ++j) v.v[j] += y.v[j] * pinv * to_f(w.v[j]);
+      } else {
+        const F y = result(ch);
+#pragma unroll
+        for (int j = 0; j < V; ++j) v.v[j] += y.v[j];
+      }
+      *reinterpret_cast<F*>(x + (size_t)t * width + ch) = v;
     }
-    xs[ch] = v;
-    ss = fmaf(v, v, ss);
+    *reinterpret_cast<F*>(xs + ch) = v;
+#pragma unroll
+    for (int j = 0; j < V; ++j) ss = fmaf(v.v[j], v.v[j], ss);
   }
+  auto out = [&](AT* row, int ch, float f, const WT* w) {
+    const F v = *reinterpret_cast<const F*>(xs + ch);
+    VecN<AT, V> o;
+#pragma unroll
+    for (int j = 0; j < V; ++j) o.v[j] = from_f<AT>(w ? v.v[j] * f * to_f(w[ch + j]) : v.v[j]);
+    *reinterpret_cast<VecN<AT, V>*>(row + ch) = o;
+  };
   if (c.cast_out)
-    for (int ch = threadIdx.x; ch < width; ch += blockDim.x) ((AT*)c.cast_out)[(size_t)t * c.ld_cast + ch] = from_f<AT>(xs[ch]);
+    for (int ch = first; ch < width; ch += step) out((AT*)c.cast_out + (size_t)t * c.ld_cast, ch, 1.0f, nullptr);
   if (!c.norm_w) return;
-  ss = block_sum(ss, red);
-  const float inv = 1.0f / sqrtf(ss / (float)width + c.eps);
-  for (int ch = threadIdx.x; ch < width; ch += blockDim.x)
-    h[(size_t)t * width + ch] = from_f<AT>(xs[ch] * inv * to_f(((const WT*)c.norm_w)[ch]));
+  const float inv = 1.0f / sqrtf(block_sum(ss, red) / (float)width + c.eps);
+  for (int ch = first; ch < width; ch += step) out(h + (size_t)t * width, ch, inv, (const WT*)c.norm_w);
 }
 
 // The embedding output x0 into the second half of the loop projection's operand [T, 2 width].
