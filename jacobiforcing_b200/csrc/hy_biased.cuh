@@ -333,19 +333,19 @@ __global__ void __launch_bounds__(128) biased_attn_kernel(Batch b, const AT* __r
 // operands, fp32 accumulators); scale, cap, distance bias and the online softmax in fp32; O += P V with P split into a
 // bf16 head and a bf16 remainder (the weights stay 32-bit in effect).  The sink joins the denominator at the end.  Key and
 // value rows are zero-padded to DP columns in shared memory (dim, vdim multiples of 8, at most DP); key / value tiles are
-// double buffered (STAGES = 2), or single buffered where there are more units than SMs: half the shared memory lets two blocks
-// share an SM and hide each other's copies.  With n_splits > 1 (steps of few rows, decoding) a unit's tile list is cut into n_splits runs, each run
+// double buffered.  PLAIN: no cap, no bias, no kept first tokens, every key up to the row's position seen; tiles that all rows see in
+// full skip the mask.  With n_splits > 1 (steps of few rows, decoding) a unit's tile list is cut into n_splits runs, each run
 // leaves (maximum, denominator, unnormalised output) per row, and biased_combine_kernel merges them with the sink.  tanh and the logarithm use the fast exponential / logarithm units: 1 - 2 / (exp(2 z) + 1) and
 // log(1 + r2 d), both far inside the rounding of the bf16 operands.
-template <int DP, int STAGES>
+template <int DP, bool PLAIN>
 __global__ void __launch_bounds__(128) biased_mma_kernel(Batch b, const AttnUnit* __restrict__ units, const bf16* __restrict__ q,
                                                          int ldq, BiasedCfg c, const bf16* __restrict__ kc,
                                                          const bf16* __restrict__ vc, bf16* __restrict__ out, int ldo,
                                                          int n_splits, float* __restrict__ part_o, float* __restrict__ part_ml) {
   constexpr int LD = DP + 8;                            // padded row (elements): ldmatrix rows fall into distinct banks
   extern __shared__ __align__(16) unsigned char hy_smem[];
-  bf16* kbuf = reinterpret_cast<bf16*>(hy_smem);        // [STAGES][64 * LD] key tiles: one in use, one in flight
-  bf16* vbuf = kbuf + STAGES * 64 * LD;                 // [STAGES][64 * LD] value tiles; the query tile sits in the first one at the start
+  bf16* kbuf = reinterpret_cast<bf16*>(hy_smem);        // [2][64 * LD] key tiles: one in use, one in flight
+  bf16* vbuf = kbuf + 2 * 64 * LD;                      // [2][64 * LD] value tiles; the query tile sits in the first one at the start
   const AttnUnit u = units[blockIdx.x];
   const int R = c.H / c.G;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
@@ -389,11 +389,11 @@ __global__ void __launch_bounds__(128) biased_mma_kernel(Batch b, const AttnUnit
   const int n_keep_tiles = min((c.keep + 63) / 64, tok0 / 64);                                  // kept tiles before it
   const int n_tiles = n_keep_tiles + (p_last / 64 - tok0 / 64 + 1);
   auto tile_j0 = [&](int it) { return it < n_keep_tiles ? it * 64 : tok0 + (it - n_keep_tiles) * 64; };
-  // copies of tile `it` into buffer it % STAGES (asynchronous; rows beyond the last position and columns beyond the head size are zeros)
+  // copies of tile `it` into buffer it & 1 (asynchronous; rows beyond the last position and columns beyond the head size are zeros)
   auto load_tile = [&](int it) {
     const int j0 = tile_j0(it);
-    bf16* ks = kbuf + (it % STAGES) * 64 * LD;
-    bf16* vs = vbuf + (it % STAGES) * 64 * LD;
+    bf16* ks = kbuf + (it & 1) * 64 * LD;
+    bf16* vs = vbuf + (it & 1) * 64 * LD;
     for (int i = tid; i < 64 * (DP / 8); i += 128) {
       const int r = i / (DP / 8), ch = i % (DP / 8);
       const int j = j0 + r;
@@ -413,13 +413,12 @@ __global__ void __launch_bounds__(128) biased_mma_kernel(Batch b, const AttnUnit
     it_lo = min(u.split * per, n_tiles);
     it_hi = min(it_lo + per, n_tiles);
   }
-  if (STAGES > 1 && it_lo < it_hi) load_tile(it_lo);
+  if (it_lo < it_hi) load_tile(it_lo);
   for (int it = it_lo; it < it_hi; ++it) {
     const int j0 = tile_j0(it);
-    const bf16* ks = kbuf + (it % STAGES) * 64 * LD;
-    const bf16* vs = vbuf + (it % STAGES) * 64 * LD;
-    if (STAGES == 1) { load_tile(it); jf::cp_async_wait_all(); }
-    else if (it + 1 < it_hi) { load_tile(it + 1); jf::cp_async_wait_1(); }         // the next tile flies under this tile's products
+    const bf16* ks = kbuf + (it & 1) * 64 * LD;
+    const bf16* vs = vbuf + (it & 1) * 64 * LD;
+    if (it + 1 < it_hi) { load_tile(it + 1); jf::cp_async_wait_1(); }         // the next tile flies under this tile's products
     else jf::cp_async_wait_all();
     __syncthreads();
     if (warp_live) {
@@ -439,6 +438,30 @@ __global__ void __launch_bounds__(128) biased_mma_kernel(Batch b, const AttnUnit
       }
     }
     float mx_lo = -INFINITY, mx_hi = -INFINITY;
+    if (PLAIN && j0 + 63 <= p_first) {
+#pragma unroll
+      for (int nb = 0; nb < 8; ++nb) {
+#pragma unroll
+        for (int cc = 0; cc < 2; ++cc) {
+          s[nb][cc] *= c.scale;
+          s[nb][2 + cc] *= c.scale;
+          mx_lo = fmaxf(mx_lo, s[nb][cc]);
+          mx_hi = fmaxf(mx_hi, s[nb][2 + cc]);
+        }
+      }
+    } else if (PLAIN) {
+#pragma unroll
+      for (int nb = 0; nb < 8; ++nb) {
+#pragma unroll
+        for (int cc = 0; cc < 2; ++cc) {
+          const int j = j0 + nb * 8 + (lane & 3) * 2 + cc;
+          s[nb][cc] = j <= p_lo ? s[nb][cc] * c.scale : -INFINITY;
+          s[nb][2 + cc] = j <= p_hi ? s[nb][2 + cc] * c.scale : -INFINITY;
+          mx_lo = fmaxf(mx_lo, s[nb][cc]);
+          mx_hi = fmaxf(mx_hi, s[nb][2 + cc]);
+        }
+      }
+    } else {
 #pragma unroll
     for (int nb = 0; nb < 8; ++nb) {
 #pragma unroll
@@ -463,6 +486,7 @@ __global__ void __launch_bounds__(128) biased_mma_kernel(Batch b, const AttnUnit
         mx_lo = fmaxf(mx_lo, s[nb][cc]);
         mx_hi = fmaxf(mx_hi, s[nb][2 + cc]);
       }
+    }
     }
     mx_lo = fmaxf(mx_lo, __shfl_xor_sync(0xffffffffu, mx_lo, 1));
     mx_lo = fmaxf(mx_lo, __shfl_xor_sync(0xffffffffu, mx_lo, 2));

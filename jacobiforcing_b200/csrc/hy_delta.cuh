@@ -6,8 +6,9 @@
 // Both dot products are taken over the state as the token finds it, side by side:
 //   p = S^T k, r = S^T q ;  u = beta (v - g p) ;  o = g r + (k.q) u ;  S <- g S + k u^T
 // so a token costs one pass over the state, one exchange between lanes and one update.  Value columns are independent of each
-// other, so a head is cut into blocks of 128 / PARTS columns that run side by side on different SMs, and PARTS lanes share a
-// column, each holding DR / PARTS of its key rows in registers (the layout of gla_kernel).
+// other, so a head is cut into blocks of 256 / PARTS columns that run side by side on different SMs, and PARTS lanes share a
+// pair of columns, each holding DR / PARTS of their key rows in registers (the layout of gla_kernel).  The next token's rows
+// are read from shared memory while the current token's dot products travel between lanes.
 #pragma once
 #include "hy_kernels.cuh"
 #include "hy_mixers.cuh"
@@ -77,7 +78,7 @@ __global__ void __launch_bounds__(128) key_value_prep_kernel(Batch b, AT* __rest
 __host__ __device__ constexpr int delta_tb(int dr) { return dr <= 128 ? 32 : dr <= 256 ? 16 : dr <= 512 ? 8 : 4; }
 template <typename AT>
 __host__ __device__ constexpr size_t delta_head_smem(int dr, int parts) {
-  const size_t tb = (size_t)delta_tb(dr), cpb = 128 / (size_t)parts, d2 = 2 * (size_t)dr;
+  const size_t tb = (size_t)delta_tb(dr), cpb = 256 / (size_t)parts, d2 = 2 * (size_t)dr;
   return (tb * (d2 + cpb + 4)) * 4 + 2 * tb * (d2 + (cpb < 8 ? 8 : cpb)) * sizeof(AT);
 }
 
@@ -91,7 +92,7 @@ __global__ void __launch_bounds__(128) delta_head_kernel(Batch b, const AT* __re
                                                          const float* __restrict__ dt_bias, int H, int G, int dim, int vdim,
                                                          int blocks_per_head, int async_ok, float* __restrict__ state,
                                                          float* __restrict__ o, int ldo) {
-  constexpr int TB = delta_tb(DR), RP = DR / PARTS, CW = 32 / PARTS, CPB = 4 * CW, CH = 16 / (int)sizeof(AT);
+  constexpr int TB = delta_tb(DR), RP = DR / PARTS, CW = 32 / PARTS, CPB = 8 * CW, CH = 16 / (int)sizeof(AT);
   constexpr int RW = 2 * DR + (CPB < 8 ? 8 : CPB);
   extern __shared__ __align__(16) unsigned char hy_smem[];
   float* sq = reinterpret_cast<float*>(hy_smem);               // [TB][DR] unit queries times dim^(-1/2)
@@ -102,16 +103,16 @@ __global__ void __launch_bounds__(128) delta_head_kernel(Batch b, const AT* __re
   const int h = blockIdx.x / blocks_per_head, c0 = (blockIdx.x % blocks_per_head) * CPB, e = blockIdx.y;
   const int g = h / (H / G);
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
-  const int cl = warp * CW + lane % CW, part = lane / CW, col = c0 + cl;
+  const int cl = 2 * (warp * CW + lane % CW), part = lane / CW, col = c0 + cl;
   const int ncol = min(CPB, vdim - c0);
-  const bool live = col < vdim;
   const int start = b.ent_start[e], cnt = b.ent_start[e + 1] - start, pos0 = b.ent_pos0[e];
   float* st = state + ((size_t)b.ent_slot[e] * H + h) * dim * vdim;
-  float S[RP];
+  float S[2][RP];
 #pragma unroll
   for (int i = 0; i < RP; ++i) {
     const int r = 4 * (part + PARTS * (i / 4)) + (i & 3);
-    S[i] = (live && r < dim && pos0 > 0) ? st[(size_t)r * vdim + col] : 0.0f;
+#pragma unroll
+    for (int c = 0; c < 2; ++c) S[c][i] = (col + c < vdim && r < dim && pos0 > 0) ? st[(size_t)r * vdim + col + c] : 0.0f;
   }
   const float rate = expf(A_log[h]), bias = dt_bias[h], qscale = 1.0f / sqrtf((float)dim);
   const bool ahead = async_ok && cnt > 1;
@@ -148,6 +149,7 @@ __global__ void __launch_bounds__(128) delta_head_kernel(Batch b, const AT* __re
       scf[4 * tid] = expf(-rate * softplus_f(ba[t * ldba + H + h] + bias));
       scf[4 * tid + 1] = sigmoid_f(ba[t * ldba + h]);
     }
+#pragma unroll 2
     for (int tt = warp; tt < nb; tt += 4) {
       constexpr int EL = (DR + 31) / 32;
       const size_t t = (size_t)(start + j0 + tt);
@@ -177,41 +179,67 @@ __global__ void __launch_bounds__(128) delta_head_kernel(Batch b, const AT* __re
     __syncthreads();
     if (ahead && j0 + TB < cnt) fetch(j0 + TB, min(TB, cnt - j0 - TB), buf ^ 1);     // that buffer was read before the barrier above
     float* po = o + (size_t)(start + j0) * ldo + h * vdim + col;
-    float keep = 0.0f;                                         // lane `part` keeps the read-out of token tt = part (mod PARTS)
-#pragma unroll 2
-    for (int tt = 0; tt < nb; ++tt) {
+    float keep0 = 0.0f, keep1 = 0.0f;                          // lane `part` keeps the read-outs of token tt = part (mod PARTS)
+    float k[RP], q[RP];
+    float4 s; float2 v;
+    auto rows = [&](int tt) {
       const float4* k4 = reinterpret_cast<const float4*>(sk + tt * DR) + part;
       const float4* q4 = reinterpret_cast<const float4*>(sq + tt * DR) + part;
-      const float4 s = sc[tt];
-      const float v = sv[tt * CPB + cl];
-      float kr[RP];
-      float p0 = 0.0f, p1 = 0.0f, p2 = 0.0f, p3 = 0.0f, r0 = 0.0f, r1 = 0.0f, r2 = 0.0f, r3 = 0.0f;
 #pragma unroll
       for (int i = 0; i < RP / 4; ++i) {
-        const float4 k = k4[i * PARTS], q = q4[i * PARTS];
-        kr[4 * i] = k.x; kr[4 * i + 1] = k.y; kr[4 * i + 2] = k.z; kr[4 * i + 3] = k.w;
-        p0 = fmaf(S[4 * i], k.x, p0);     r0 = fmaf(S[4 * i], q.x, r0);
-        p1 = fmaf(S[4 * i + 1], k.y, p1); r1 = fmaf(S[4 * i + 1], q.y, r1);
-        p2 = fmaf(S[4 * i + 2], k.z, p2); r2 = fmaf(S[4 * i + 2], q.z, r2);
-        p3 = fmaf(S[4 * i + 3], k.w, p3); r3 = fmaf(S[4 * i + 3], q.w, r3);
+        const float4 kk = k4[i * PARTS], qq = q4[i * PARTS];
+        k[4 * i] = kk.x; k[4 * i + 1] = kk.y; k[4 * i + 2] = kk.z; k[4 * i + 3] = kk.w;
+        q[4 * i] = qq.x; q[4 * i + 1] = qq.y; q[4 * i + 2] = qq.z; q[4 * i + 3] = qq.w;
       }
-      float p = (p0 + p1) + (p2 + p3), r = (r0 + r1) + (r2 + r3);
+      s = sc[tt];
+      v = *reinterpret_cast<const float2*>(sv + tt * CPB + cl);
+    };
+    rows(0);
+    for (int tt = 0; tt < nb; ++tt) {
+      // values 0, 1: S^T k of both columns, 2, 3: S^T q
+      float d[4] = {0.0f, 0.0f, 0.0f, 0.0f}, f[4] = {0.0f, 0.0f, 0.0f, 0.0f};
 #pragma unroll
-      for (int x = CW; x < 32; x <<= 1) { p += __shfl_xor_sync(0xffffffffu, p, x); r += __shfl_xor_sync(0xffffffffu, r, x); }
-      const float u = s.y * fmaf(-s.x, p, v);
+      for (int i = 0; i < RP; i += 2) {
 #pragma unroll
-      for (int i = 0; i < RP; ++i) S[i] = fmaf(s.x, S[i], kr[i] * u);
-      if ((tt & (PARTS - 1)) == part) keep = fmaf(s.z, u, s.x * r);
-      if (((tt & (PARTS - 1)) == PARTS - 1 || tt == nb - 1) && live && part <= (tt & (PARTS - 1)))
-        po[(size_t)((tt & ~(PARTS - 1)) + part) * ldo] = keep;
+        for (int c = 0; c < 2; ++c) {
+          d[c] = fmaf(S[c][i], k[i], d[c]);     f[c] = fmaf(S[c][i + 1], k[i + 1], f[c]);
+          d[2 + c] = fmaf(S[c][i], q[i], d[2 + c]); f[2 + c] = fmaf(S[c][i + 1], q[i + 1], f[2 + c]);
+        }
+      }
+      float kc[RP];
+      const float4 sn = s;
+      const float2 vn = v;
+#pragma unroll
+      for (int i = 0; i < RP; ++i) kc[i] = k[i];
+      if (tt + 1 < nb) rows(tt + 1);
+#pragma unroll
+      for (int c = 0; c < 4; ++c) d[c] += f[c];
+#pragma unroll
+      for (int x = CW; x < 32; x <<= 1) {
+#pragma unroll
+        for (int c = 0; c < 4; ++c) d[c] += __shfl_xor_sync(0xffffffffu, d[c], x);
+      }
+      const float u0 = sn.y * fmaf(-sn.x, d[0], vn.x), u1 = sn.y * fmaf(-sn.x, d[1], vn.y);
+#pragma unroll
+      for (int i = 0; i < RP; ++i) {
+        S[0][i] = fmaf(sn.x, S[0][i], kc[i] * u0);
+        S[1][i] = fmaf(sn.x, S[1][i], kc[i] * u1);
+      }
+      const int slot = tt & (PARTS - 1);
+      if (slot == part) { keep0 = fmaf(sn.z, u0, sn.x * d[2]); keep1 = fmaf(sn.z, u1, sn.x * d[3]); }
+      if ((slot == PARTS - 1 || tt == nb - 1) && part <= slot) {
+        float* row = po + (size_t)(tt - slot + part) * ldo;
+        if (col < vdim) row[0] = keep0;
+        if (col + 1 < vdim) row[1] = keep1;
+      }
     }
   }
-  if (live) {
 #pragma unroll
-    for (int i = 0; i < RP; ++i) {
-      const int r = 4 * (part + PARTS * (i / 4)) + (i & 3);
-      if (r < dim) st[(size_t)r * vdim + col] = S[i];
-    }
+  for (int i = 0; i < RP; ++i) {
+    const int r = 4 * (part + PARTS * (i / 4)) + (i & 3);
+#pragma unroll
+    for (int c = 0; c < 2; ++c)
+      if (col + c < vdim && r < dim) st[(size_t)r * vdim + col + c] = S[c][i];
   }
 }
 

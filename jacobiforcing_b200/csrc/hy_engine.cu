@@ -2196,15 +2196,21 @@ void biased_attend(hy_engine* h, const Batch& b, const LayerW& L, const hy_layer
         tc = true;
         static bool attr = false;
         if (!attr) {
-          cudaFuncSetAttribute(biased_mma_kernel<64, 2>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)window_mma_smem(64));
-          cudaFuncSetAttribute(biased_mma_kernel<128, 1>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)window_mma_smem(128) / 2);
-          cudaFuncSetAttribute(biased_mma_kernel<128, 2>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)window_mma_smem(128));
+          cudaFuncSetAttribute(biased_mma_kernel<64, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)window_mma_smem(64));
+          cudaFuncSetAttribute(biased_mma_kernel<64, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)window_mma_smem(64));
+          cudaFuncSetAttribute(biased_mma_kernel<128, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)window_mma_smem(128));
+          cudaFuncSetAttribute(biased_mma_kernel<128, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)window_mma_smem(128));
           attr = true;
         }
 #define HY_BIASED_ARGS b, u->d, pin + L.c_q, h->ld_pin, bc, (const bf16*)L.cache, (const bf16*)L.cache_v, cat, h->ld_cat, u->ns, h->part_o, h->part_ml
-        if (dp == 64) biased_mma_kernel<64, 2><<<u->n, 128, window_mma_smem(64), s>>>(HY_BIASED_ARGS);
-        else if (u->n > 148) biased_mma_kernel<128, 1><<<u->n, 128, window_mma_smem(128) / 2, s>>>(HY_BIASED_ARGS);
-        else biased_mma_kernel<128, 2><<<u->n, 128, window_mma_smem(128), s>>>(HY_BIASED_ARGS);
+        const bool pl = bc.bias == HY_BIAS_NONE && bc.cap <= 0.0f && !bc.window && !bc.keep && !bc.chunk;
+        if (dp == 64) {
+          if (pl) biased_mma_kernel<64, true><<<u->n, 128, window_mma_smem(64), s>>>(HY_BIASED_ARGS);
+          else biased_mma_kernel<64, false><<<u->n, 128, window_mma_smem(64), s>>>(HY_BIASED_ARGS);
+        } else {
+          if (pl) biased_mma_kernel<128, true><<<u->n, 128, window_mma_smem(128), s>>>(HY_BIASED_ARGS);
+          else biased_mma_kernel<128, false><<<u->n, 128, window_mma_smem(128), s>>>(HY_BIASED_ARGS);
+        }
 #undef HY_BIASED_ARGS
         if (u->ns > 1) {
           biased_combine_kernel<bf16><<<T * c.b_heads, 64, 0, s>>>(h->part_o, h->part_ml, bc, dp, u->ns, cat, h->ld_cat);
@@ -2321,7 +2327,7 @@ void gla_mixer(hy_engine* h, const Batch& b, const LayerW& L, const hy_layer_cfg
   ProfScope ps(h, HY_PROF_DELTA);
   const int ch = 16 / (int)sizeof(AT);
   auto launch = [&](auto kern, int parts, size_t smem) {
-    const int cpb = 128 / parts, bph = (dv + cpb - 1) / cpb;
+    const int cpb = 256 / parts, bph = (dv + cpb - 1) / cpb;
     const int async_ok = (dk % ch == 0 && dk % 4 == 0 && dv % ch == 0 && cpb % ch == 0 && h->ld_pin % ch == 0 && L.c_k % ch == 0 && L.c_v % ch == 0) ? 1 : 0;
     cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     kern<<<dim3(H * bph, E), 128, smem, s>>>(b, pin, h->ld_pin, L.c_q, L.c_k, L.c_v, h->f2, h->ld_f2, H, dk, dv, bph, async_ok, L.rec_state,
@@ -2329,9 +2335,9 @@ void gla_mixer(hy_engine* h, const Batch& b, const LayerW& L, const hy_layer_cfg
   };
   if (dk <= 16) launch(gla_kernel<AT, 16, 4>, 4, gla_smem<AT>(16, 4));
   else if (dk <= 32) launch(gla_kernel<AT, 32, 4>, 4, gla_smem<AT>(32, 4));
-  else if (dk <= 64) launch(gla_kernel<AT, 64, 4>, 4, gla_smem<AT>(64, 4));
-  else if (dk <= 128) launch(gla_kernel<AT, 128, 8>, 8, gla_smem<AT>(128, 8));
-  else if (dk <= 256) launch(gla_kernel<AT, 256, 16>, 16, gla_smem<AT>(256, 16));
+  else if (dk <= 64) launch(gla_kernel<AT, 64, 8>, 8, gla_smem<AT>(64, 8));
+  else if (dk <= 128) launch(gla_kernel<AT, 128, 16>, 16, gla_smem<AT>(128, 16));
+  else if (dk <= 256) launch(gla_kernel<AT, 256, 32>, 32, gla_smem<AT>(256, 32));
   else if (dk <= 512) launch(gla_kernel<AT, 512, 32>, 32, gla_smem<AT>(512, 32));
   else launch(gla_kernel<AT, 1024, 32>, 32, gla_smem<AT>(1024, 32));
   gla_out_kernel<AT><<<(T * H + 3) / 4, 128, 0, s>>>(T, H, dv, h->f2 + c_o, h->ld_f2, pin + L.c_g, h->ld_pin, L.g_norm, h->m.norm_eps,
@@ -2350,7 +2356,7 @@ void retention_mixer(hy_engine* h, const Batch& b, const LayerW& L, const hy_lay
   ProfScope ps(h, HY_PROF_DELTA);
   const int ch = 16 / (int)sizeof(AT);
   auto launch = [&](auto kern, int parts, size_t smem) {
-    const int cpb = 128 / parts, bph = (dv + cpb - 1) / cpb;
+    const int cpb = 256 / parts, bph = (dv + cpb - 1) / cpb;
     const int async_ok = (dk % ch == 0 && dv % ch == 0 && cpb % ch == 0 && h->ld_pin % ch == 0 && L.c_k % ch == 0 && L.c_v % ch == 0) ? 1 : 0;
     cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     kern<<<dim3(H * bph, E), 128, smem, s>>>(b, pin, h->ld_pin, L.c_q, L.c_k, L.c_v, rot.out, rot.ld, H, dk, dv, bph, async_ok, L.rec_state,
@@ -2358,9 +2364,9 @@ void retention_mixer(hy_engine* h, const Batch& b, const LayerW& L, const hy_lay
   };
   if (dk <= 16) launch(gla_kernel<AT, 16, 4, true>, 4, gla_smem<AT>(16, 4));
   else if (dk <= 32) launch(gla_kernel<AT, 32, 4, true>, 4, gla_smem<AT>(32, 4));
-  else if (dk <= 64) launch(gla_kernel<AT, 64, 4, true>, 4, gla_smem<AT>(64, 4));
-  else if (dk <= 128) launch(gla_kernel<AT, 128, 8, true>, 8, gla_smem<AT>(128, 8));
-  else if (dk <= 256) launch(gla_kernel<AT, 256, 16, true>, 16, gla_smem<AT>(256, 16));
+  else if (dk <= 64) launch(gla_kernel<AT, 64, 8, true>, 8, gla_smem<AT>(64, 8));
+  else if (dk <= 128) launch(gla_kernel<AT, 128, 16, true>, 16, gla_smem<AT>(128, 16));
+  else if (dk <= 256) launch(gla_kernel<AT, 256, 32, true>, 32, gla_smem<AT>(256, 32));
   else if (dk <= 512) launch(gla_kernel<AT, 512, 32, true>, 32, gla_smem<AT>(512, 32));
   else launch(gla_kernel<AT, 1024, 32, true>, 32, gla_smem<AT>(1024, 32));
   gla_out_kernel<AT><<<(T * H + 3) / 4, 128, 0, s>>>(T, H, dv, h->f2, h->ld_f2, pin + L.c_g, h->ld_pin, nullptr, h->m.norm_eps, 1.0f, cat,
@@ -2393,7 +2399,7 @@ void attn_delta_mixer(hy_engine* h, const Batch& b, const LayerW& L, const hy_la
   ProfScope ps(h, HY_PROF_DELTA);
   const int ch = 16 / (int)sizeof(AT);
   auto launch = [&](auto kern, int parts, size_t smem) {
-    const int cpb = 128 / parts, bph = (dv + cpb - 1) / cpb;
+    const int cpb = 256 / parts, bph = (dv + cpb - 1) / cpb;
     const int async_ok = (dk % ch == 0 && dv % ch == 0 && cpb % ch == 0 && h->ld_cv % ch == 0) ? 1 : 0;
     cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     kern<<<dim3(H * bph, E), 128, smem, s>>>(b, cv, h->ld_cv, 0, nk, 2 * nk, h->f1 + c.b_heads, h->ld_f1, (const float*)L.A_log,
@@ -2401,9 +2407,9 @@ void attn_delta_mixer(hy_engine* h, const Batch& b, const LayerW& L, const hy_la
   };
   if (dk <= 16) launch(delta_head_kernel<AT, 16, 4>, 4, delta_head_smem<AT>(16, 4));
   else if (dk <= 32) launch(delta_head_kernel<AT, 32, 4>, 4, delta_head_smem<AT>(32, 4));
-  else if (dk <= 64) launch(delta_head_kernel<AT, 64, 4>, 4, delta_head_smem<AT>(64, 4));
-  else if (dk <= 128) launch(delta_head_kernel<AT, 128, 8>, 8, delta_head_smem<AT>(128, 8));
-  else if (dk <= 256) launch(delta_head_kernel<AT, 256, 16>, 16, delta_head_smem<AT>(256, 16));
+  else if (dk <= 64) launch(delta_head_kernel<AT, 64, 8>, 8, delta_head_smem<AT>(64, 8));
+  else if (dk <= 128) launch(delta_head_kernel<AT, 128, 16>, 16, delta_head_smem<AT>(128, 16));
+  else if (dk <= 256) launch(delta_head_kernel<AT, 256, 32>, 32, delta_head_smem<AT>(256, 32));
   else if (dk <= 512) launch(delta_head_kernel<AT, 512, 32>, 32, delta_head_smem<AT>(512, 32));
   else launch(delta_head_kernel<AT, 1024, 32>, 32, delta_head_smem<AT>(1024, 32));
   gla_out_kernel<AT><<<(T * H + 3) / 4, 128, 0, s>>>(T, H, dv, h->f2, h->ld_f2, pin + L.c_g, h->ld_pin, L.g_norm, h->m.norm_eps,

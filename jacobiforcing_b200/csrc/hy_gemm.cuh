@@ -4,8 +4,9 @@
 // Swap-AB like the Jacobi engine's GEMMs: the WEIGHT tile is the MMA's A operand (M = 128 output features, so the
 // accumulator's lanes are features and a warp's epilogue stores are contiguous along n), the token rows are the B operand
 // (N = BT tokens, 128 or 256).  Weights are stored in HBM already in the K-major SWIZZLE_128B tile layout (one contiguous
-// 16 KiB tile per 128 features x 64 k: one bulk copy per pipeline stage, no tensor map); the activation tile is read
-// row-major with 16-byte loads by four producer warps that write it swizzled into shared memory.
+// 16 KiB tile per 128 features x 64 k: one bulk copy per pipeline stage, no tensor map); the activation tile travels
+// row-major by asynchronous 16-byte copies of four producer warps, each copy to its swizzled place in shared memory.  The
+// copies of all stages but one are in flight at any time; a thread hands a stage over once its own copies have landed.
 //
 // Warps 0-3: activation producers, then the epilogue (TMEM -> registers -> global, through GemmOut).
 // Warp 4:    weight producer (one lane, cp.async.bulk + mbarrier expect_tx).
@@ -17,12 +18,13 @@
 
 namespace hy {
 
-constexpr int TC_STAGES = 4;
+constexpr int TC_MAX_STAGES = 4;
+__host__ __device__ constexpr int tc_stages(int bt) { return 2; }   // three (two) blocks per SM: their prologues and epilogues overlap other blocks' products
 constexpr int TC_WTILE = 128 * 64 * 2;                 // 16 KiB
 constexpr uint32_t TC_SPIN_LIMIT = 1u << 22;           // try_wait probes (each blocks for a bounded time itself)
 
 struct TcSmem {
-  uint64_t full[TC_STAGES], empty[TC_STAGES], acc_full;
+  uint64_t full[TC_MAX_STAGES], empty[TC_MAX_STAGES], acc_full;
   uint32_t tmem_base;
   uint32_t failed;
 };
@@ -51,6 +53,7 @@ __global__ void __launch_bounds__(192) gemm_tc_kernel(const bf16* __restrict__ X
                                                       int N, int K, GemmOut o, int* err, TcGroup grp) {
   extern __shared__ __align__(16) unsigned char hy_smem[];
   unsigned char* base = reinterpret_cast<unsigned char*>((reinterpret_cast<uintptr_t>(hy_smem) + 1023) & ~(uintptr_t)1023);
+  constexpr int TC_STAGES = tc_stages(BT);
   constexpr int XTILE = BT * 128;                        // BT rows of 64 bf16
   constexpr int SLOT = TC_WTILE + XTILE;
   TcSmem* sm = reinterpret_cast<TcSmem*>(base + TC_STAGES * SLOT);
@@ -84,27 +87,28 @@ __global__ void __launch_bounds__(192) gemm_tc_kernel(const bf16* __restrict__ X
       const int t = t0 + ((threadIdx.x + u * 128) >> 3);
       srow[u] = t < T ? (grp.row_map ? grp.row_map[t] : t) : -1;
     }
-    for (int kt = 0; kt < KT; ++kt) {
-      const int s = kt % TC_STAGES;
-      unsigned char* xt = base + s * SLOT + TC_WTILE;
-      // all loads of the stage first (BT / 16 independent 16-byte loads per thread in flight), then the swizzled stores
-      uint4 v[BT / 16];
+    constexpr int AHEAD = TC_STAGES - 1;                  // stages in flight behind the one that is handed over
+    for (int kt = 0; kt < KT + AHEAD; ++kt) {
+      if (kt < KT) {
+        const int s = kt % TC_STAGES;
+        unsigned char* xt = base + s * SLOT + TC_WTILE;
+        if (!tc_wait(&sm->empty[s], ((kt / TC_STAGES) & 1) ^ 1, sm, err)) break;   // the slot is free: MMAs that read it retired
 #pragma unroll
-      for (int u = 0; u < BT / 16; ++u) {
-        const int k = kt * 64 + ((threadIdx.x + u * 128) & 7) * 8;
-        v[u] = make_uint4(0, 0, 0, 0);
-        if (srow[u] >= 0 && k < K) v[u] = *reinterpret_cast<const uint4*>(X + (size_t)srow[u] * lda + k);
+        for (int u = 0; u < BT / 16; ++u) {
+          const int i = threadIdx.x + u * 128;
+          const int r = i >> 3, c = i & 7, k = kt * 64 + c * 8;
+          const bool ok = srow[u] >= 0 && k < K;          // rows and columns beyond the operand are zeros
+          jf::cp_async_16(xt + r * 128 + ((c ^ (r & 7)) << 4), ok ? X + (size_t)srow[u] * lda + k : X, ok ? 16u : 0u);
+        }
       }
-      if (!tc_wait(&sm->empty[s], ((kt / TC_STAGES) & 1) ^ 1, sm, err)) break;     // the slot is free: MMAs that read it retired
-#pragma unroll
-      for (int u = 0; u < BT / 16; ++u) {
-        const int i = threadIdx.x + u * 128;
-        const int r = i >> 3, c = i & 7;
-        *reinterpret_cast<uint4*>(xt + r * 128 + ((c ^ (r & 7)) << 4)) = v[u];
+      jf::cp_async_commit();                              // one group per turn, empty ones behind the last stage
+      if (kt >= AHEAD) {
+        jf::cp_async_wait<AHEAD>();                       // this thread's copies of stage kt - AHEAD have landed
+        jf::fence_proxy_async_smem();
+        jf::mbar_arrive(&sm->full[(kt - AHEAD) % TC_STAGES]);
       }
-      jf::fence_proxy_async_smem();
-      jf::mbar_arrive(&sm->full[s]);
     }
+    jf::cp_async_wait_all();
     // ---- epilogue ----------------------------------------------------------------------------------------------------
     if (tc_wait(&sm->acc_full, 0, sm, err)) {
       jf::tc_fence_after();
@@ -174,7 +178,7 @@ __global__ void __launch_bounds__(192) gemm_tc_kernel(const bf16* __restrict__ X
   if (warp == 5) jf::tmem_dealloc(sm->tmem_base, BT);
 }
 
-constexpr size_t tc_smem_bytes(int bt) { return (size_t)TC_STAGES * (TC_WTILE + bt * 128) + sizeof(TcSmem) + 1024; }
+constexpr size_t tc_smem_bytes(int bt) { return (size_t)tc_stages(bt) * (TC_WTILE + bt * 128) + sizeof(TcSmem) + 1024; }
 
 // Host-side packer: row-major [N, K] floats -> bf16 tiles [ceil(N/128)][ceil(K/64)] of 128 x 64 in the swizzled layout.
 inline void pack_tiles(const float* w, int N, int K, std::vector<uint16_t>& out) {

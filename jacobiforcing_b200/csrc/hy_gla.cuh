@@ -8,8 +8,9 @@
 // recurrence) and no weight in the norm.
 //
 // The recurrence has no feedback from the read-out and its value columns are independent, so a head is cut into blocks of
-// CPB = 128 / PARTS columns that run side by side on different SMs, and PARTS lanes share a column, each holding DR / PARTS
-// of its key rows in registers.  The norm needs whole heads: it follows in a kernel of its own (gla_out_kernel).
+// CPB = 256 / PARTS columns that run side by side on different SMs; PARTS lanes share a pair of columns, each holding DR / PARTS
+// of their key rows in registers (two columns per lane: the rows read from shared memory per token, which bound the kernel with
+// one column per lane, serve twice the work).  The norm needs whole heads: it follows in a kernel of its own (gla_out_kernel).
 #pragma once
 #include "hy_kernels.cuh"
 #include "hy_delta.cuh"
@@ -21,14 +22,14 @@ namespace hy {
 __host__ __device__ constexpr int gla_tb(int dr) { return dr <= 128 ? 32 : dr <= 256 ? 16 : dr <= 512 ? 8 : 4; }
 template <typename AT>
 __host__ __device__ constexpr size_t gla_smem(int dr, int parts) {
-  const size_t tb = (size_t)gla_tb(dr), cpb = 128 / (size_t)parts, d2 = 2 * (size_t)dr;
+  const size_t tb = (size_t)gla_tb(dr), cpb = 256 / (size_t)parts, d2 = 2 * (size_t)dr;
   // fp32 rows q, k | values; two buffers of raw q, k, v rows (values padded to 16 bytes) and of decays in flight
   return (tb * (d2 + cpb)) * 4 + 2 * tb * ((d2 + (cpb < 8 ? 8 : cpb)) * sizeof(AT) + (size_t)dr * 4);
 }
 
 // in [T, ld]: q at col_q, k at col_k (heads * dim each), v at col_v (heads * vdim).  decay [T, ldd] fp32 (heads * dim).
 // o [T, ldo] fp32 (heads * vdim).  state [slot][H][dim][vdim] fp32.  grid (H * blocks_per_head, entries), 128 threads.
-// Lane layout: column = warp * (32 / PARTS) + lane % (32 / PARTS), part = lane / (32 / PARTS); part r holds the key rows
+// Lane layout: columns 2 c, 2 c + 1 with c = warp * (32 / PARTS) + lane % (32 / PARTS), part = lane / (32 / PARTS); part r holds the key rows
 // 4 (r + PARTS i) .. + 3, so the PARTS row quadruples a warp reads from shared memory at once lie next to each other.
 // async_ok: head sizes, leading dimensions and column offsets are multiples of 16 bytes, and so is CPB: raw rows of the next batch of tokens travel by asynchronous
 // copies while the current batch runs; short entries (decode steps) and odd sizes stage directly.
@@ -39,7 +40,7 @@ __global__ void __launch_bounds__(128) gla_kernel(Batch b, const AT* __restrict_
                                                   const float* __restrict__ decay, int ldd, int H, int dim, int vdim,
                                                   int blocks_per_head, int async_ok, float* __restrict__ state,
                                                   float* __restrict__ o, int ldo, const float* __restrict__ head_decay, RotPair rp) {
-  constexpr int TB = gla_tb(DR), RP = DR / PARTS, CW = 32 / PARTS, CPB = 4 * CW, CH = 16 / (int)sizeof(AT);
+  constexpr int TB = gla_tb(DR), RP = DR / PARTS, CW = 32 / PARTS, CPB = 8 * CW, CH = 16 / (int)sizeof(AT);
   extern __shared__ __align__(16) unsigned char hy_smem[];
   float* sq = reinterpret_cast<float*>(hy_smem);               // [TB][DR] scaled queries
   float* sk = sq + TB * DR;                                    // [TB][DR] keys
@@ -49,16 +50,16 @@ __global__ void __launch_bounds__(128) gla_kernel(Batch b, const AT* __restrict_
   AT* raw = reinterpret_cast<AT*>(sa + 2 * TB * DR);           // [2][TB][RW] raw q | k | v rows in flight
   const int h = blockIdx.x / blocks_per_head, c0 = (blockIdx.x % blocks_per_head) * CPB, e = blockIdx.y;
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
-  const int cl = warp * CW + lane % CW, part = lane / CW, col = c0 + cl;
+  const int cl = 2 * (warp * CW + lane % CW), part = lane / CW, col = c0 + cl;
   const int ncol = min(CPB, vdim - c0);
-  const bool live = col < vdim;
   const int start = b.ent_start[e], cnt = b.ent_start[e + 1] - start, pos0 = b.ent_pos0[e];
   float* st = state + ((size_t)b.ent_slot[e] * H + h) * dim * vdim;
-  float S[RP];
+  float S[2][RP];
 #pragma unroll
   for (int i = 0; i < RP; ++i) {
     const int r = 4 * (part + PARTS * (i / 4)) + (i & 3);
-    S[i] = (live && r < dim && pos0 > 0) ? st[(size_t)r * vdim + col] : 0.0f;
+#pragma unroll
+    for (int c = 0; c < 2; ++c) S[c][i] = (col + c < vdim && r < dim && pos0 > 0) ? st[(size_t)r * vdim + col + c] : 0.0f;
   }
   const float qscale = 1.0f / sqrtf((float)dim);
   const bool ahead = async_ok && cnt > 1;
@@ -96,23 +97,29 @@ __global__ void __launch_bounds__(128) gla_kernel(Batch b, const AT* __restrict_
       for (int i = tid; i < 2 * TB * DR; i += 128) if (i % DR >= dim) sa[i] = 0.0f;
     fetch(0, min(TB, cnt), 0);
   }
-  // one token's update of this lane's key rows; returns its part of the read-out
-  auto update = [&](const float* ca, int tt) {
+  // one token's update of this lane's key rows; leaves its part of both columns' read-outs in p[0], p[1]
+  auto update = [&](const float* ca, int tt, float* p) {
     const float4* a4 = reinterpret_cast<const float4*>(ca + tt * DR) + part;
     const float4* k4 = reinterpret_cast<const float4*>(sk + tt * DR) + part;
     const float4* q4 = reinterpret_cast<const float4*>(sq + tt * DR) + part;
-    const float v = sv[tt * CPB + cl];
-    float p0 = 0.0f, p1 = 0.0f, p2 = 0.0f, p3 = 0.0f;
+    const float2 v2 = *reinterpret_cast<const float2*>(sv + tt * CPB + cl);
+    float x[2] = {0.0f, 0.0f}, y[2] = {0.0f, 0.0f};
 #pragma unroll
     for (int i = 0; i < RP / 4; ++i) {
       const float4 k = k4[i * PARTS], q = q4[i * PARTS];
       const float4 a = ROT ? make_float4(hd, hd, hd, hd) : a4[i * PARTS];
-      S[4 * i] = fmaf(a.x, S[4 * i], k.x * v);         p0 = fmaf(S[4 * i], q.x, p0);
-      S[4 * i + 1] = fmaf(a.y, S[4 * i + 1], k.y * v); p1 = fmaf(S[4 * i + 1], q.y, p1);
-      S[4 * i + 2] = fmaf(a.z, S[4 * i + 2], k.z * v); p2 = fmaf(S[4 * i + 2], q.z, p2);
-      S[4 * i + 3] = fmaf(a.w, S[4 * i + 3], k.w * v); p3 = fmaf(S[4 * i + 3], q.w, p3);
+#pragma unroll
+      for (int c = 0; c < 2; ++c) {
+        const float v = c ? v2.y : v2.x;
+        float* R = &S[c][4 * i];
+        R[0] = fmaf(a.x, R[0], k.x * v); x[c] = fmaf(R[0], q.x, x[c]);
+        R[1] = fmaf(a.y, R[1], k.y * v); y[c] = fmaf(R[1], q.y, y[c]);
+        R[2] = fmaf(a.z, R[2], k.z * v); x[c] = fmaf(R[2], q.z, x[c]);
+        R[3] = fmaf(a.w, R[3], k.w * v); y[c] = fmaf(R[3], q.w, y[c]);
+      }
     }
-    return (p0 + p1) + (p2 + p3);
+    p[0] = x[0] + y[0];
+    p[1] = x[1] + y[1];
   };
   constexpr int TG = TB < 8 ? TB : 8;                          // tokens whose read-outs are reduced together
   int buf = 0;
@@ -201,18 +208,19 @@ __global__ void __launch_bounds__(128) gla_kernel(Batch b, const AT* __restrict_
     float* po = o + (size_t)(start + j0) * ldo + h * vdim + col;
     int tt = 0;
     for (; tt + TG <= nb; tt += TG) {
-      // TG tokens without a shuffle between them, then one exchange in which every step halves the tokens a lane keeps
-      float p[TG];
+      // TG tokens without a shuffle between them, then one exchange in which every step halves the values a lane keeps
+      constexpr int VT = 2 * TG;                               // value 2 u + c: token tt + u, column col + c
+      float p[VT];
 #pragma unroll
-      for (int u = 0; u < TG; ++u) p[u] = update(ca, tt + u);
-      int n = TG, base = 0;
+      for (int u = 0; u < TG; ++u) update(ca, tt + u, p + 2 * u);
+      int n = VT, base = 0;
 #pragma unroll
       for (int s = 16; s >= CW; s >>= 1) {
         const bool hi = (lane & s) != 0;
         if (n > 1) {
           n >>= 1;
 #pragma unroll
-          for (int u = 0; u < TG / 2; ++u) {
+          for (int u = 0; u < VT / 2; ++u) {
             if (u >= n) break;
             const float other = __shfl_xor_sync(0xffffffffu, hi ? p[u] : p[u + n], s);
             p[u] = (hi ? p[u + n] : p[u]) + other;
@@ -222,25 +230,32 @@ __global__ void __launch_bounds__(128) gla_kernel(Batch b, const AT* __restrict_
           p[0] += __shfl_xor_sync(0xffffffffu, p[0], s);
         }
       }
-      constexpr int LEFT = TG > PARTS ? TG / PARTS : 1, SAME = PARTS > TG ? PARTS / TG : 1;     // tokens per lane, lanes per token
-      if (live && (part & (SAME - 1)) == 0) {
+      constexpr int LEFT = VT > PARTS ? VT / PARTS : 1, SAME = PARTS > VT ? PARTS / VT : 1;     // values per lane, lanes per value
+      if ((part & (SAME - 1)) == 0) {
 #pragma unroll
-        for (int u = 0; u < LEFT; ++u) po[(size_t)(tt + base + u) * ldo] = p[u];
+        for (int u = 0; u < LEFT; ++u) {
+          const int c = (base + u) & 1;
+          if (col + c < vdim) po[(size_t)(tt + (base + u) / 2) * ldo + c] = p[u];
+        }
       }
     }
     for (; tt < nb; ++tt) {
-      float p = update(ca, tt);
+      float p[2];
+      update(ca, tt, p);
 #pragma unroll
-      for (int s = CW; s < 32; s <<= 1) p += __shfl_xor_sync(0xffffffffu, p, s);
-      if (live && part == 0) po[(size_t)tt * ldo] = p;
+      for (int s = CW; s < 32; s <<= 1) {
+        p[0] += __shfl_xor_sync(0xffffffffu, p[0], s);
+        p[1] += __shfl_xor_sync(0xffffffffu, p[1], s);
+      }
+      if (part < 2 && col + part < vdim) po[(size_t)tt * ldo + part] = part ? p[1] : p[0];
     }
   }
-  if (live) {
 #pragma unroll
-    for (int i = 0; i < RP; ++i) {
-      const int r = 4 * (part + PARTS * (i / 4)) + (i & 3);
-      if (r < dim) st[(size_t)r * vdim + col] = S[i];
-    }
+  for (int i = 0; i < RP; ++i) {
+    const int r = 4 * (part + PARTS * (i / 4)) + (i & 3);
+#pragma unroll
+    for (int c = 0; c < 2; ++c)
+      if (col + c < vdim && r < dim) st[(size_t)r * vdim + col + c] = S[c][i];
   }
 }
 
