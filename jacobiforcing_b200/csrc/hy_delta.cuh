@@ -6,9 +6,11 @@
 // Both dot products are taken over the state as the token finds it, side by side:
 //   p = S^T k, r = S^T q ;  u = beta (v - g p) ;  o = g r + (k.q) u ;  S <- g S + k u^T
 // so a token costs one pass over the state, one exchange between lanes and one update.  Value columns are independent of each
-// other, so a head is cut into blocks of 256 / PARTS columns that run side by side on different SMs, and PARTS lanes share a
-// pair of columns, each holding DR / PARTS of their key rows in registers (the layout of gla_kernel).  The next token's rows
-// are read from shared memory while the current token's dot products travel between lanes.
+// other, so a head is cut into blocks of 128 / PARTS columns that run side by side on different SMs, and PARTS lanes share a
+// column, each holding DR / PARTS of its key rows in registers.  With one warp per scheduler the recurrence runs at about a
+// third of the issue rate whatever the layout, so its time is its instruction count: everything that does not depend on the
+// state (convolutions, unit vectors, k.q, decays, step sizes; rotations) is made beforehand, once per token and key head, by
+// kernels of their own that leave fp32 rows, and the recurrence copies those asynchronously.
 #pragma once
 #include "hy_kernels.cuh"
 #include "hy_mixers.cuh"
@@ -73,173 +75,214 @@ __global__ void __launch_bounds__(128) key_value_prep_kernel(Batch b, AT* __rest
   }
 }
 
-// ---- gated delta rule, one decay per head ---------------------------------------------------------------------------------------------
-// tokens staged per batch and shared memory: fp32 rows q, k | values | 3 scalars per token; two buffers of raw q, k, v rows
-__host__ __device__ constexpr int delta_tb(int dr) { return dr <= 128 ? 32 : dr <= 256 ? 16 : dr <= 512 ? 8 : 4; }
+// ---- operands of a matrix-state recurrence: fp32 rows [T][heads][q dim | k dim] ------------------------------------------------------
+// Rotated (rp.pairs > 0: the first 2 pairs dimensions, cs [T, ldc] from rot_tables_kernel), queries times dim^(-1/2).
 template <typename AT>
-__host__ __device__ constexpr size_t delta_head_smem(int dr, int parts) {
-  const size_t tb = (size_t)delta_tb(dr), cpb = 256 / (size_t)parts, d2 = 2 * (size_t)dr;
-  return (tb * (d2 + cpb + 4)) * 4 + 2 * tb * (d2 + (cpb < 8 ? 8 : cpb)) * sizeof(AT);
+__global__ void __launch_bounds__(1024) linear_rows_kernel(const AT* __restrict__ in, int ld, int col_q, int col_k, int H, int dim,
+                                                          const float* __restrict__ cs, int ldc, RotPair rp, float* __restrict__ qk) {
+  const int t = blockIdx.x;
+  const AT* row = in + (size_t)t * ld;
+  const float* c = rp.pairs > 0 ? cs + (size_t)t * ldc : nullptr;
+  float* out = qk + (size_t)t * H * 2 * dim;
+  const float qscale = 1.0f / sqrtf((float)dim);
+  for (int i = threadIdx.x; i < H * dim; i += blockDim.x) {
+    const int h = i / dim, k = i % dim;
+    const AT* qh = row + col_q + h * dim;
+    const AT* kh = row + col_k + h * dim;
+    float q = to_f(qh[k]), kk = to_f(kh[k]);
+    if (k < 2 * rp.pairs) {
+      const int p = rp.partner(k);
+      q = rp.turn(c, k, q, to_f(qh[p]));
+      kk = rp.turn(c, k, kk, to_f(kh[p]));
+    }
+    out[(size_t)h * 2 * dim + k] = q * qscale;
+    out[(size_t)h * 2 * dim + dim + k] = kk;
+  }
 }
 
-// in [T, ld] (after convolution and activation): q at col_q, k at col_k (G heads of dim each), v at col_v (H heads of vdim).
-// ba [T, ldba] fp32: step-size pre-activations at column h, decay pre-activations at column H + h.
-// o [T, ldo] fp32 (H heads of vdim), before the output norm.  state [slot][H][dim][vdim] fp32.
-// grid (H * blocks_per_head, entries), 128 threads; lane layout and async_ok as in gla_kernel.
-template <typename AT, int DR, int PARTS>
-__global__ void __launch_bounds__(128) delta_head_kernel(Batch b, const AT* __restrict__ in, int ld, int col_q, int col_k, int col_v,
+// The delta rule's: causal convolution over time with silu of the columns [q (G heads of dim) | k | v (H heads of vdim)] at col0
+// (see conv_kernel: w [C, taps], state [slot][taps - 1][C]), values into v [T, ldv] in the activation type, queries and keys made
+// unit vectors per head, and per head (decay, step size, k.q) into sc [T][H].  ba [T, ldba] fp32: step-size pre-activations at
+// column h, decay pre-activations at column H + h.  One block per token.
+template <typename AT, typename WT>
+__global__ void __launch_bounds__(1024) delta_rows_kernel(Batch b, const AT* __restrict__ u, int ldu, int col0, int H, int G, int dim, int vdim,
+                                                         int taps, const WT* __restrict__ w, const float* __restrict__ state,
                                                          const float* __restrict__ ba, int ldba, const float* __restrict__ A_log,
-                                                         const float* __restrict__ dt_bias, int H, int G, int dim, int vdim,
-                                                         int blocks_per_head, int async_ok, float* __restrict__ state,
-                                                         float* __restrict__ o, int ldo) {
-  constexpr int TB = delta_tb(DR), RP = DR / PARTS, CW = 32 / PARTS, CPB = 8 * CW, CH = 16 / (int)sizeof(AT);
-  constexpr int RW = 2 * DR + (CPB < 8 ? 8 : CPB);
+                                                         const float* __restrict__ dt_bias, AT* __restrict__ v, int ldv,
+                                                         float* __restrict__ qk, float4* __restrict__ sc) {
   extern __shared__ __align__(16) unsigned char hy_smem[];
-  float* sq = reinterpret_cast<float*>(hy_smem);               // [TB][DR] unit queries times dim^(-1/2)
-  float* sk = sq + TB * DR;                                    // [TB][DR] unit keys
-  float* sv = sk + TB * DR;                                    // [TB][CPB] values
-  float4* sc = reinterpret_cast<float4*>(sv + TB * CPB);       // [TB] decay, step size, k.q
-  AT* raw = reinterpret_cast<AT*>(sc + TB);                    // [2][TB][RW] raw q | k | v rows in flight
+  float* row = reinterpret_cast<float*>(hy_smem);              // [2 G dim] convolved queries, then keys
+  const int t = blockIdx.x, e = b.tok_ent[t];
+  const int start = b.ent_start[e], pos0 = b.ent_pos0[e], j = t - start;
+  const int nk = G * dim, C = 2 * nk + H * vdim;
+  const float* st = state + (size_t)b.ent_slot[e] * (taps - 1) * C;
+  for (int c = threadIdx.x; c < C; c += blockDim.x) {
+    float acc = 0.0f;
+    for (int i = 0; i < taps; ++i) {
+      const int src = j - (taps - 1) + i;
+      float x = 0.0f;
+      if (src >= 0) x = to_f(u[(size_t)(start + src) * ldu + col0 + c]);
+      else if (pos0 + src >= 0) x = st[(size_t)(taps - 1 + src) * C + c];
+      acc = fmaf(to_f(w[(size_t)c * taps + i]), x, acc);
+    }
+    acc = silu_f(acc);
+    if (c < 2 * nk) row[c] = acc;
+    else v[(size_t)t * ldv + c - 2 * nk] = from_f<AT>(acc);
+  }
+  __syncthreads();
+  const int lane = threadIdx.x & 31, R = H / G;
+  const float qscale = 1.0f / sqrtf((float)dim);
+  for (int g = threadIdx.x >> 5; g < G; g += blockDim.x >> 5) {
+    const float* qr = row + g * dim;
+    const float* kr = row + nk + g * dim;
+    float q2 = 0.0f, k2 = 0.0f, kq = 0.0f;
+    for (int k = lane; k < dim; k += 32) { q2 = fmaf(qr[k], qr[k], q2); k2 = fmaf(kr[k], kr[k], k2); kq = fmaf(qr[k], kr[k], kq); }
+    q2 = warp_sum(q2); k2 = warp_sum(k2); kq = warp_sum(kq);
+    const float qi = qscale / sqrtf(q2 + 1e-6f), ki = 1.0f / sqrtf(k2 + 1e-6f);
+    float* out = qk + ((size_t)t * G + g) * 2 * dim;
+    for (int k = lane; k < dim; k += 32) { out[k] = qr[k] * qi; out[dim + k] = kr[k] * ki; }
+    for (int r = lane; r < R; r += 32) {
+      const int h = g * R + r;
+      const float decay = expf(-expf(A_log[h]) * softplus_f(ba[(size_t)t * ldba + H + h] + dt_bias[h]));
+      sc[(size_t)t * H + h] = make_float4(decay, sigmoid_f(ba[(size_t)t * ldba + h]), kq * qi * ki, 0.0f);
+    }
+  }
+}
+
+// ---- staging shared by the recurrences -----------------------------------------------------------------------------------------------
+// tokens per batch; two buffers of fp32 rows q | k (DR each, zero beyond dim) and of value rows in the activation type
+__host__ __device__ constexpr int lin_tb(int dr) { return dr <= 128 ? 32 : dr <= 256 ? 16 : dr <= 512 ? 8 : 4; }
+__host__ __device__ constexpr int lin_cpb(int parts) { return 128 / parts; }
+template <typename AT>
+__host__ __device__ constexpr size_t lin_smem(int dr, int parts, int more_floats) {      // more_floats: per token, beside q and k
+  return 2 * (size_t)lin_tb(dr) * ((2 * (size_t)dr + more_floats) * 4 + (lin_cpb(parts) < 8 ? 8 : lin_cpb(parts)) * sizeof(AT));
+}
+
+// n floats of each of nb rows (row r at src + r * ld) to dst + r * dld: asynchronous 16-byte copies where everything is aligned
+__device__ __forceinline__ void copy_rows(float* dst, int dld, const float* src, size_t ld, int nb, int n, bool vec) {
+  if (vec) {
+    const int nc = n / 4;
+    for (int i = threadIdx.x; i < nb * nc; i += 128) {
+      const int r = i / nc, c = i % nc * 4;
+      jf::cp_async_16(dst + r * dld + c, src + (size_t)r * ld + c, 16u);
+    }
+  } else {
+    for (int i = threadIdx.x; i < nb * n; i += 128) dst[i / n * dld + i % n] = src[(size_t)(i / n) * ld + i % n];
+  }
+}
+template <typename AT>
+__device__ __forceinline__ void copy_values(AT* dst, int dld, const AT* src, size_t ld, int nb, int n, bool vec) {
+  constexpr int CH = 16 / (int)sizeof(AT);
+  if (vec) {
+    const int nc = n / CH;
+    for (int i = threadIdx.x; i < nb * nc; i += 128) {
+      const int r = i / nc, c = i % nc * CH;
+      jf::cp_async_16(dst + r * dld + c, src + (size_t)r * ld + c, 16u);
+    }
+  } else {
+    for (int i = threadIdx.x; i < nb * n; i += 128) dst[i / n * dld + i % n] = src[(size_t)(i / n) * ld + i % n];
+  }
+}
+
+// ---- gated delta rule, one decay per head ---------------------------------------------------------------------------------------------
+// qk [T][G][q dim | k dim] and sc [T][H] from delta_rows_kernel, v [T, ldv] (H heads of vdim).  o [T, ldo] fp32 (H heads of vdim),
+// before the output norm.  state [slot][H][dim][vdim] fp32.  grid (H * blocks_per_head, entries), 128 threads.
+// Lane layout: column = warp * (32 / PARTS) + lane % (32 / PARTS), part = lane / (32 / PARTS); part r holds the key rows
+// 4 (r + PARTS i) .. + 3, so the PARTS row quadruples a warp reads from shared memory at once lie next to each other.  vec: key
+// rows are multiples of 16 bytes; vvec: a block's value rows are.
+template <typename AT, int DR, int PARTS>
+__global__ void __launch_bounds__(128) delta_head_kernel(Batch b, const float* __restrict__ qk, const AT* __restrict__ v, int ldv,
+                                                         const float4* __restrict__ scal, int H, int G, int dim, int vdim,
+                                                         int blocks_per_head, int vec, int vvec, float* __restrict__ state,
+                                                         float* __restrict__ o, int ldo) {
+  constexpr int TB = lin_tb(DR), RP = DR / PARTS, CW = 32 / PARTS, CPB = lin_cpb(PARTS), VW = CPB < 8 ? 8 : CPB;
+  extern __shared__ __align__(16) unsigned char hy_smem[];
+  float* sqk = reinterpret_cast<float*>(hy_smem);              // [2][TB][2 DR]
+  float4* ssc = reinterpret_cast<float4*>(sqk + 2 * TB * 2 * DR);      // [2][TB]
+  AT* sv = reinterpret_cast<AT*>(ssc + 2 * TB);                // [2][TB][VW]
   const int h = blockIdx.x / blocks_per_head, c0 = (blockIdx.x % blocks_per_head) * CPB, e = blockIdx.y;
   const int g = h / (H / G);
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
-  const int cl = 2 * (warp * CW + lane % CW), part = lane / CW, col = c0 + cl;
+  const int cl = warp * CW + lane % CW, part = lane / CW, col = c0 + cl;
   const int ncol = min(CPB, vdim - c0);
+  const bool live = col < vdim;
   const int start = b.ent_start[e], cnt = b.ent_start[e + 1] - start, pos0 = b.ent_pos0[e];
   float* st = state + ((size_t)b.ent_slot[e] * H + h) * dim * vdim;
-  float S[2][RP];
+  float S[RP];
 #pragma unroll
   for (int i = 0; i < RP; ++i) {
     const int r = 4 * (part + PARTS * (i / 4)) + (i & 3);
-#pragma unroll
-    for (int c = 0; c < 2; ++c) S[c][i] = (col + c < vdim && r < dim && pos0 > 0) ? st[(size_t)r * vdim + col + c] : 0.0f;
+    S[i] = (live && r < dim && pos0 > 0) ? st[(size_t)r * vdim + col] : 0.0f;
   }
-  const float rate = expf(A_log[h]), bias = dt_bias[h], qscale = 1.0f / sqrtf((float)dim);
-  const bool ahead = async_ok && cnt > 1;
-  const AT* inq = in + col_q + g * dim;
-  const AT* ink = in + col_k + g * dim;
-  const AT* inv = in + col_v + h * vdim + c0;
-  auto fetch = [&](int j0, int nb, int buf) {
-    AT* dst = raw + (size_t)buf * TB * RW;
+  if (dim < DR)                                                // rows beyond the head's key size stay zero
+    for (int i = tid; i < 2 * TB * 2 * DR; i += 128) if (i % DR >= dim) sqk[i] = 0.0f;
+  auto fetch = [&](int j0, int buf) {
+    const int nb = min(TB, cnt - j0);
     const size_t t0 = (size_t)(start + j0);
-    constexpr int QC = DR / CH, VC = CPB >= CH ? CPB / CH : 1;
-    for (int i = tid; i < nb * QC; i += 128) {
-      const int tt = i / QC, k = i % QC * CH;
-      if (k >= dim) continue;
-      jf::cp_async_16(dst + (size_t)tt * RW + k, inq + (t0 + tt) * ld + k, 16u);
-      jf::cp_async_16(dst + (size_t)tt * RW + DR + k, ink + (t0 + tt) * ld + k, 16u);
-    }
-    for (int i = tid; i < nb * VC; i += 128) {
-      const int tt = i / VC, k = i % VC * CH;
-      if (k < ncol) jf::cp_async_16(dst + (size_t)tt * RW + 2 * DR + k, inv + (t0 + tt) * ld + k, 16u);
-    }
+    float* d = sqk + (size_t)buf * TB * 2 * DR;
+    const float* src = qk + (t0 * G + g) * 2 * dim;
+    const size_t ld = (size_t)G * 2 * dim;
+    copy_rows(d, 2 * DR, src, ld, nb, dim, vec);
+    copy_rows(d + DR, 2 * DR, src + dim, ld, nb, dim, vec);
+    if (tid < nb) jf::cp_async_16(ssc + buf * TB + tid, scal + (t0 + tid) * H + h, 16u);
+    copy_values(sv + (size_t)buf * TB * VW, VW, v + t0 * ldv + h * vdim + c0, ldv, nb, ncol, vvec);
     jf::cp_async_commit();
   };
-  if (ahead) fetch(0, min(TB, cnt), 0);
+  fetch(0, 0);
   int buf = 0;
   for (int j0 = 0; j0 < cnt; j0 += TB, buf ^= 1) {
     const int nb = min(TB, cnt - j0);
-    if (ahead) jf::cp_async_wait_all();
-    __syncthreads();                                           // raw rows have landed; the previous batch is finished
-    const AT* src = raw + (size_t)buf * TB * RW;
-    // decays and step sizes: one thread per token; unit vectors and k.q: one warp per token
-    float* scf = reinterpret_cast<float*>(sc);
-    if (tid < nb) {
-      const size_t t = (size_t)(start + j0 + tid);
-      scf[4 * tid] = expf(-rate * softplus_f(ba[t * ldba + H + h] + bias));
-      scf[4 * tid + 1] = sigmoid_f(ba[t * ldba + h]);
-    }
-#pragma unroll 2
-    for (int tt = warp; tt < nb; tt += 4) {
-      constexpr int EL = (DR + 31) / 32;
-      const size_t t = (size_t)(start + j0 + tt);
-      float qv[EL], kv[EL];
-      float q2 = 0.0f, k2 = 0.0f, qk = 0.0f;
-#pragma unroll
-      for (int i = 0; i < EL; ++i) {
-        const int k = lane + 32 * i;
-        const bool ok = k < dim;
-        qv[i] = ok ? to_f(ahead ? src[(size_t)tt * RW + k] : inq[t * ld + k]) : 0.0f;
-        kv[i] = ok ? to_f(ahead ? src[(size_t)tt * RW + DR + k] : ink[t * ld + k]) : 0.0f;
-        q2 = fmaf(qv[i], qv[i], q2); k2 = fmaf(kv[i], kv[i], k2); qk = fmaf(qv[i], kv[i], qk);
-      }
-      q2 = warp_sum(q2); k2 = warp_sum(k2); qk = warp_sum(qk);
-      const float qi = qscale / sqrtf(q2 + 1e-6f), ki = 1.0f / sqrtf(k2 + 1e-6f);
-#pragma unroll
-      for (int i = 0; i < EL; ++i) {
-        const int k = lane + 32 * i;
-        if (k < DR) { sq[tt * DR + k] = qv[i] * qi; sk[tt * DR + k] = kv[i] * ki; }
-      }
-      if (lane == 0) scf[4 * tt + 2] = qk * qi * ki;
-    }
-    for (int i = tid; i < nb * CPB; i += 128) {
-      const int tt = i / CPB, k = i % CPB;
-      sv[i] = k < ncol ? to_f(ahead ? src[(size_t)tt * RW + 2 * DR + k] : inv[(size_t)(start + j0 + tt) * ld + k]) : 0.0f;
-    }
-    __syncthreads();
-    if (ahead && j0 + TB < cnt) fetch(j0 + TB, min(TB, cnt - j0 - TB), buf ^ 1);     // that buffer was read before the barrier above
+    jf::cp_async_wait_all();
+    __syncthreads();                                           // this batch has landed; the batch before it is finished
+    if (j0 + TB < cnt) fetch(j0 + TB, buf ^ 1);
+    const float* qb = sqk + (size_t)buf * TB * 2 * DR + 4 * part;
+    const AT* vb = sv + (size_t)buf * TB * VW + min(cl, ncol - 1);
     float* po = o + (size_t)(start + j0) * ldo + h * vdim + col;
-    float keep0 = 0.0f, keep1 = 0.0f;                          // lane `part` keeps the read-outs of token tt = part (mod PARTS)
-    float k[RP], q[RP];
-    float4 s; float2 v;
+    float keep = 0.0f;                                         // lane `part` keeps the read-out of token tt = part (mod PARTS)
+    float k[RP], q[RP], vv;
+    float4 s;
     auto rows = [&](int tt) {
-      const float4* k4 = reinterpret_cast<const float4*>(sk + tt * DR) + part;
-      const float4* q4 = reinterpret_cast<const float4*>(sq + tt * DR) + part;
 #pragma unroll
       for (int i = 0; i < RP / 4; ++i) {
-        const float4 kk = k4[i * PARTS], qq = q4[i * PARTS];
-        k[4 * i] = kk.x; k[4 * i + 1] = kk.y; k[4 * i + 2] = kk.z; k[4 * i + 3] = kk.w;
+        const float4 qq = *reinterpret_cast<const float4*>(qb + tt * 2 * DR + 4 * PARTS * i);
+        const float4 kk = *reinterpret_cast<const float4*>(qb + tt * 2 * DR + DR + 4 * PARTS * i);
         q[4 * i] = qq.x; q[4 * i + 1] = qq.y; q[4 * i + 2] = qq.z; q[4 * i + 3] = qq.w;
+        k[4 * i] = kk.x; k[4 * i + 1] = kk.y; k[4 * i + 2] = kk.z; k[4 * i + 3] = kk.w;
       }
-      s = sc[tt];
-      v = *reinterpret_cast<const float2*>(sv + tt * CPB + cl);
+      s = ssc[buf * TB + tt];
+      vv = to_f(vb[tt * VW]);
     };
     rows(0);
+#pragma unroll 2
     for (int tt = 0; tt < nb; ++tt) {
-      // values 0, 1: S^T k of both columns, 2, 3: S^T q
-      float d[4] = {0.0f, 0.0f, 0.0f, 0.0f}, f[4] = {0.0f, 0.0f, 0.0f, 0.0f};
+      float p0 = 0.0f, p1 = 0.0f, r0 = 0.0f, r1 = 0.0f, kc[RP];
 #pragma unroll
       for (int i = 0; i < RP; i += 2) {
-#pragma unroll
-        for (int c = 0; c < 2; ++c) {
-          d[c] = fmaf(S[c][i], k[i], d[c]);     f[c] = fmaf(S[c][i + 1], k[i + 1], f[c]);
-          d[2 + c] = fmaf(S[c][i], q[i], d[2 + c]); f[2 + c] = fmaf(S[c][i + 1], q[i + 1], f[2 + c]);
-        }
+        p0 = fmaf(S[i], k[i], p0); p1 = fmaf(S[i + 1], k[i + 1], p1);
+        r0 = fmaf(S[i], q[i], r0); r1 = fmaf(S[i + 1], q[i + 1], r1);
       }
-      float kc[RP];
+      float p = p0 + p1, r = r0 + r1;
       const float4 sn = s;
-      const float2 vn = v;
+      const float vn = vv;
 #pragma unroll
       for (int i = 0; i < RP; ++i) kc[i] = k[i];
-      if (tt + 1 < nb) rows(tt + 1);
+      rows(min(tt + 1, nb - 1));                               // the next token's rows fly under the exchange
 #pragma unroll
-      for (int c = 0; c < 4; ++c) d[c] += f[c];
+      for (int x = CW; x < 32; x <<= 1) { p += __shfl_xor_sync(0xffffffffu, p, x); r += __shfl_xor_sync(0xffffffffu, r, x); }
+      const float u = sn.y * fmaf(-sn.x, p, vn);
 #pragma unroll
-      for (int x = CW; x < 32; x <<= 1) {
-#pragma unroll
-        for (int c = 0; c < 4; ++c) d[c] += __shfl_xor_sync(0xffffffffu, d[c], x);
-      }
-      const float u0 = sn.y * fmaf(-sn.x, d[0], vn.x), u1 = sn.y * fmaf(-sn.x, d[1], vn.y);
-#pragma unroll
-      for (int i = 0; i < RP; ++i) {
-        S[0][i] = fmaf(sn.x, S[0][i], kc[i] * u0);
-        S[1][i] = fmaf(sn.x, S[1][i], kc[i] * u1);
-      }
+      for (int i = 0; i < RP; ++i) S[i] = fmaf(sn.x, S[i], kc[i] * u);
       const int slot = tt & (PARTS - 1);
-      if (slot == part) { keep0 = fmaf(sn.z, u0, sn.x * d[2]); keep1 = fmaf(sn.z, u1, sn.x * d[3]); }
-      if ((slot == PARTS - 1 || tt == nb - 1) && part <= slot) {
-        float* row = po + (size_t)(tt - slot + part) * ldo;
-        if (col < vdim) row[0] = keep0;
-        if (col + 1 < vdim) row[1] = keep1;
-      }
+      if (slot == part) keep = fmaf(sn.z, u, sn.x * r);
+      if ((slot == PARTS - 1 || tt == nb - 1) && live && part <= slot) po[(size_t)(tt - slot + part) * ldo] = keep;
     }
   }
+  if (live) {
 #pragma unroll
-  for (int i = 0; i < RP; ++i) {
-    const int r = 4 * (part + PARTS * (i / 4)) + (i & 3);
-#pragma unroll
-    for (int c = 0; c < 2; ++c)
-      if (col + c < vdim && r < dim) st[(size_t)r * vdim + col + c] = S[c][i];
+    for (int i = 0; i < RP; ++i) {
+      const int r = 4 * (part + PARTS * (i / 4)) + (i & 3);
+      if (r < dim) st[(size_t)r * vdim + col] = S[i];
+    }
   }
 }
 

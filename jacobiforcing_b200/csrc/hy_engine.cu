@@ -148,6 +148,7 @@ struct hy_engine {
   bool finalized = false;
   // workspace
   float* x = nullptr; void* hbuf = nullptr; void* pin = nullptr; void* cat = nullptr; void* cv = nullptr;
+  float* lin = nullptr; float4* lin_sc = nullptr;   // fp32 operand rows and per-head scalars of a matrix-state recurrence
   float* f1 = nullptr; float* f2 = nullptr; void* hw = nullptr; float* logits = nullptr; int* sampled = nullptr;
   float* temp_d = nullptr;
   int ld_pin = 0, ld_cat = 0, ld_cv = 0, ld_f1 = 0, ld_f2 = 0;
@@ -480,7 +481,7 @@ void rotation_table(const hy_layer_cfg& c, std::vector<double>& f, float* mag) {
   }
 }
 
-struct Maxima { int in = 1, out = 1, cv = 1, f1 = 1, f2 = 1; };
+struct Maxima { int in = 1, out = 1, cv = 1, f1 = 1, f2 = 1, lin = 0, lin_sc = 0; };
 
 bool tanh_norm_load(Builder& B, const std::string& name, int W, TanhNorm* n) {
   const HostTensor* w = B.get(name, W, -1);
@@ -968,6 +969,7 @@ int finalize_parallel_layer(hy_engine* h, Builder& B, size_t i, Maxima& mx) {
     if (auto t = B.get(d + "norm", c.g_vdim, -1)) L.g_norm = B.up_f32(t->v);
     k_mix = nv;
     mx.f2 = std::max(mx.f2, ((nq + 3) & ~3) + nv);            // decays, then read-outs
+    mx.lin = std::max(mx.lin, 2 * nq);
   } else if (c.mixer == HY_MIX_BIASED) {
     const int H = c.b_heads, G = c.b_kv_heads, nq = H * c.b_dim, nk = G * c.b_dim, nv = G * c.b_vdim;
     L.c_q = 0; L.c_k = nq; L.c_v = nq + nk;
@@ -1089,6 +1091,7 @@ int finalize_rms_sandwich_layer(hy_engine* h, Builder& B, size_t i, Maxima& mx) 
     outs.push_back(B.get(d + "o", W, nv));
     if (int rc = rotation_table_of(h, B, c, L)) return rc;
     mx.f2 = std::max(mx.f2, nv);
+    mx.lin = std::max(mx.lin, 2 * nq);
     if (dev_alloc(h, (void**)&L.rec_state, (size_t)rt.num_slots * H * c.g_dim * c.g_vdim * 4, &h->bytes_state)) return HY_ERR_CUDA;
   } else if (c.mixer == HY_MIX_ATTN_DELTA) {
     const std::string a = d + "left.", r = d + "right.";
@@ -1117,8 +1120,10 @@ int finalize_rms_sandwich_layer(hy_engine* h, Builder& B, size_t i, Maxima& mx) 
     outs.push_back(B.get(a + "o", W, nq));
     outs.push_back(B.get(r + "o", W, dv));
     if (int rc = rotation_table_of(h, B, c, L)) return rc;
-    mx.cv = std::max(mx.cv, C);
+    mx.cv = std::max(mx.cv, dv);
     mx.f2 = std::max(mx.f2, dv);
+    mx.lin = std::max(mx.lin, 2 * dk);
+    mx.lin_sc = std::max(mx.lin_sc, Hd);
     if (dev_alloc(h, &L.cache, tokens * nk * h->esz(), &h->bytes_cache)) return HY_ERR_CUDA;
     if (dev_alloc(h, &L.cache_v, tokens * nk * h->esz(), &h->bytes_cache)) return HY_ERR_CUDA;
     if (dev_alloc(h, (void**)&L.conv_state, (size_t)rt.num_slots * (c.d_conv - 1) * C * 4, &h->bytes_state)) return HY_ERR_CUDA;
@@ -1321,6 +1326,8 @@ extern "C" int hy_finalize(hy_handle h) {
   if (dev_alloc(h, &h->cv, T * h->ld_cv * es, &h->bytes_ws)) return HY_ERR_CUDA;
   if (dev_alloc(h, (void**)&h->f1, T * h->ld_f1 * 4, &h->bytes_ws)) return HY_ERR_CUDA;
   if (dev_alloc(h, (void**)&h->f2, T * h->ld_f2 * 4, &h->bytes_ws)) return HY_ERR_CUDA;
+  if (mx.lin > 0 && dev_alloc(h, (void**)&h->lin, T * (size_t)mx.lin * 4, &h->bytes_ws)) return HY_ERR_CUDA;
+  if (mx.lin_sc > 0 && dev_alloc(h, (void**)&h->lin_sc, T * (size_t)mx.lin_sc * sizeof(float4), &h->bytes_ws)) return HY_ERR_CUDA;
   if (h->m.block_kind == HY_BLOCK_PRENORM) {
     if (dev_alloc(h, (void**)&h->hn, T * W * 4, &h->bytes_ws)) return HY_ERR_CUDA;
     if (h->m.depth_avg && dev_alloc(h, (void**)&h->kept, (h->lc.size() + 1) * T * W * 4, &h->bytes_ws)) return HY_ERR_CUDA;
@@ -2311,6 +2318,27 @@ int prenorm_layer(hy_engine* h, const Batch& b, size_t li) {
   return HY_OK;
 }
 
+// Register layout of a matrix-state recurrence by key size: fn(padded key size, lanes per column), both compile-time.
+template <typename AT, typename Fn>
+void launch_linear(int dk, Fn fn) {
+  if (dk <= 16) fn(std::integral_constant<int, 16>{}, std::integral_constant<int, 4>{});
+  else if (dk <= 32) fn(std::integral_constant<int, 32>{}, std::integral_constant<int, 8>{});
+  else if (dk <= 64) fn(std::integral_constant<int, 64>{}, std::integral_constant<int, 16>{});
+  else if (dk <= 128) fn(std::integral_constant<int, 128>{}, std::integral_constant<int, 16>{});
+  else if (dk <= 256) fn(std::integral_constant<int, 256>{}, std::integral_constant<int, 32>{});
+  else if (dk <= 512) fn(std::integral_constant<int, 512>{}, std::integral_constant<int, 32>{});
+  else fn(std::integral_constant<int, 1024>{}, std::integral_constant<int, 32>{});
+}
+
+// Blocks per head of a recurrence and which of its rows may travel by 16-byte copies.
+struct LinearLaunch { int bph, vec, vvec; };
+template <typename AT>
+LinearLaunch linear_launch(int parts, int dk, int dv, const AT* v, int ldv) {
+  const int cpb = lin_cpb(parts), ch = 16 / (int)sizeof(AT);
+  return LinearLaunch{(dv + cpb - 1) / cpb, dk % 4 == 0 ? 1 : 0,
+                      dv % ch == 0 && cpb % ch == 0 && ldv % ch == 0 && (reinterpret_cast<uintptr_t>(v) & 15) == 0 ? 1 : 0};
+}
+
 // Gated linear attention: projections in h->pin (q, k, v, gate), the decay's first step in h->f1; result in h->cat.
 template <typename AT>
 void gla_mixer(hy_engine* h, const Batch& b, const LayerW& L, const hy_layer_cfg& c) {
@@ -2325,24 +2353,18 @@ void gla_mixer(hy_engine* h, const Batch& b, const LayerW& L, const hy_layer_cfg
     gemm<float, WT, float>(h, h->f1, h->ld_f1, (const WT*)L.w_a2, c.g_low, T, nq, c.g_low, o);
   }
   ProfScope ps(h, HY_PROF_DELTA);
-  const int ch = 16 / (int)sizeof(AT);
-  auto launch = [&](auto kern, int parts, size_t smem) {
-    const int cpb = 256 / parts, bph = (dv + cpb - 1) / cpb;
-    const int async_ok = (dk % ch == 0 && dk % 4 == 0 && dv % ch == 0 && cpb % ch == 0 && h->ld_pin % ch == 0 && L.c_k % ch == 0 && L.c_v % ch == 0) ? 1 : 0;
-    cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-    kern<<<dim3(H * bph, E), 128, smem, s>>>(b, pin, h->ld_pin, L.c_q, L.c_k, L.c_v, h->f2, h->ld_f2, H, dk, dv, bph, async_ok, L.rec_state,
-                                             h->f2 + c_o, h->ld_f2, nullptr, RotPair{0, 1});
-  };
-  if (dk <= 16) launch(gla_kernel<AT, 16, 4>, 4, gla_smem<AT>(16, 4));
-  else if (dk <= 32) launch(gla_kernel<AT, 32, 4>, 4, gla_smem<AT>(32, 4));
-  else if (dk <= 64) launch(gla_kernel<AT, 64, 8>, 8, gla_smem<AT>(64, 8));
-  else if (dk <= 128) launch(gla_kernel<AT, 128, 16>, 16, gla_smem<AT>(128, 16));
-  else if (dk <= 256) launch(gla_kernel<AT, 256, 32>, 32, gla_smem<AT>(256, 32));
-  else if (dk <= 512) launch(gla_kernel<AT, 512, 32>, 32, gla_smem<AT>(512, 32));
-  else launch(gla_kernel<AT, 1024, 32>, 32, gla_smem<AT>(1024, 32));
+  linear_rows_kernel<AT><<<T, T <= 8 ? 1024 : 128, 0, s>>>(pin, h->ld_pin, L.c_q, L.c_k, H, dk, nullptr, 0, RotPair{0, 1}, h->lin);
+  launch_linear<AT>(dk, [&](auto dr, auto parts) {
+    constexpr int DR = decltype(dr)::value, PARTS = decltype(parts)::value;
+    const LinearLaunch g = linear_launch<AT>(PARTS, dk, dv, pin + L.c_v, h->ld_pin);
+    const size_t smem = lin_smem<AT>(DR, PARTS, DR);
+    cudaFuncSetAttribute(gla_kernel<AT, DR, PARTS, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    gla_kernel<AT, DR, PARTS, false><<<dim3(H * g.bph, E), 128, smem, s>>>(b, h->lin, pin + L.c_v, h->ld_pin, h->f2, h->ld_f2, nullptr, H, dk,
+                                                                           dv, g.bph, g.vec, g.vvec, L.rec_state, h->f2 + c_o, h->ld_f2);
+  });
   gla_out_kernel<AT><<<(T * H + 3) / 4, 128, 0, s>>>(T, H, dv, h->f2 + c_o, h->ld_f2, pin + L.c_g, h->ld_pin, L.g_norm, h->m.norm_eps,
                                                      1.0f, cat, h->ld_cat);
-  h->launches += 2;
+  h->launches += 3;
 }
 
 // Retention: projections in h->pin (q, k, v, gate); read-outs in h->f2, result in h->cat.
@@ -2354,24 +2376,18 @@ void retention_mixer(hy_engine* h, const Batch& b, const LayerW& L, const hy_lay
   const RotTable& rot = h->rot_tables[(size_t)L.rot_table].t;
   const RotPair rp{rot.pairs, c.r_half};
   ProfScope ps(h, HY_PROF_DELTA);
-  const int ch = 16 / (int)sizeof(AT);
-  auto launch = [&](auto kern, int parts, size_t smem) {
-    const int cpb = 256 / parts, bph = (dv + cpb - 1) / cpb;
-    const int async_ok = (dk % ch == 0 && dv % ch == 0 && cpb % ch == 0 && h->ld_pin % ch == 0 && L.c_k % ch == 0 && L.c_v % ch == 0) ? 1 : 0;
-    cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-    kern<<<dim3(H * bph, E), 128, smem, s>>>(b, pin, h->ld_pin, L.c_q, L.c_k, L.c_v, rot.out, rot.ld, H, dk, dv, bph, async_ok, L.rec_state,
-                                             h->f2, h->ld_f2, L.decay, rp);
-  };
-  if (dk <= 16) launch(gla_kernel<AT, 16, 4, true>, 4, gla_smem<AT>(16, 4));
-  else if (dk <= 32) launch(gla_kernel<AT, 32, 4, true>, 4, gla_smem<AT>(32, 4));
-  else if (dk <= 64) launch(gla_kernel<AT, 64, 8, true>, 8, gla_smem<AT>(64, 8));
-  else if (dk <= 128) launch(gla_kernel<AT, 128, 16, true>, 16, gla_smem<AT>(128, 16));
-  else if (dk <= 256) launch(gla_kernel<AT, 256, 32, true>, 32, gla_smem<AT>(256, 32));
-  else if (dk <= 512) launch(gla_kernel<AT, 512, 32, true>, 32, gla_smem<AT>(512, 32));
-  else launch(gla_kernel<AT, 1024, 32, true>, 32, gla_smem<AT>(1024, 32));
+  linear_rows_kernel<AT><<<T, T <= 8 ? 1024 : 128, 0, s>>>(pin, h->ld_pin, L.c_q, L.c_k, H, dk, rot.out, rot.ld, rp, h->lin);
+  launch_linear<AT>(dk, [&](auto dr, auto parts) {
+    constexpr int DR = decltype(dr)::value, PARTS = decltype(parts)::value;
+    const LinearLaunch g = linear_launch<AT>(PARTS, dk, dv, pin + L.c_v, h->ld_pin);
+    const size_t smem = lin_smem<AT>(DR, PARTS, 0);
+    cudaFuncSetAttribute(gla_kernel<AT, DR, PARTS, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    gla_kernel<AT, DR, PARTS, true><<<dim3(H * g.bph, E), 128, smem, s>>>(b, h->lin, pin + L.c_v, h->ld_pin, nullptr, 0, L.decay, H, dk, dv,
+                                                                          g.bph, g.vec, g.vvec, L.rec_state, h->f2, h->ld_f2);
+  });
   gla_out_kernel<AT><<<(T * H + 3) / 4, 128, 0, s>>>(T, H, dv, h->f2, h->ld_f2, pin + L.c_g, h->ld_pin, nullptr, h->m.norm_eps, 1.0f, cat,
                                                      h->ld_cat);
-  h->launches += 2;
+  h->launches += 3;
 }
 
 // Attention whose values are its unrotated keys beside a gated delta rule with one decay per head: operand columns in h->pin
@@ -2388,8 +2404,11 @@ void attn_delta_mixer(hy_engine* h, const Batch& b, const LayerW& L, const hy_la
     ProfScope ps(h, HY_PROF_CONV);
     key_value_prep_kernel<AT><<<T, 128, 0, s>>>(b, pin, h->ld_pin, L.c_q, L.c_k, c.b_heads, c.b_kv_heads, c.b_dim, rot.out, rot.ld,
                                                 RotPair{rot.pairs, c.r_half}, (AT*)L.cache, (AT*)L.cache_v);
-    conv_kernel<AT, WT><<<dim3((C + 127) / 128, T), 128, 0, s>>>(b, pin, h->ld_pin, L.c_x, C, c.d_conv, (const WT*)L.conv_qkv,
-                                                                 (const WT*)nullptr, 1, L.conv_state, cv, h->ld_cv);
+    static bool attr = false;                                // per AT: this function is a template
+    if (!attr) { cudaFuncSetAttribute(delta_rows_kernel<AT, WT>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024); attr = true; }
+    delta_rows_kernel<AT, WT><<<T, T <= 8 ? 1024 : 256, (size_t)2 * nk * 4, s>>>(b, pin, h->ld_pin, L.c_x, H, G, dk, dv, c.d_conv, (const WT*)L.conv_qkv,
+                                                                 L.conv_state, h->f1 + c.b_heads, h->ld_f1, (const float*)L.A_log,
+                                                                 (const float*)L.dt_bias, cv, h->ld_cv, h->lin, h->lin_sc);
     conv_tail_kernel<AT><<<dim3((C + 127) / 128, E), 128, 0, s>>>(b, pin, h->ld_pin, L.c_x, C, c.d_conv, L.conv_state);
     h->launches += 3;
   }
@@ -2397,21 +2416,14 @@ void attn_delta_mixer(hy_engine* h, const Batch& b, const LayerW& L, const hy_la
                      h->f1, h->ld_f1, c.left_scale};
   biased_attend<AT>(h, b, L, c, bc);
   ProfScope ps(h, HY_PROF_DELTA);
-  const int ch = 16 / (int)sizeof(AT);
-  auto launch = [&](auto kern, int parts, size_t smem) {
-    const int cpb = 256 / parts, bph = (dv + cpb - 1) / cpb;
-    const int async_ok = (dk % ch == 0 && dv % ch == 0 && cpb % ch == 0 && h->ld_cv % ch == 0) ? 1 : 0;
-    cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-    kern<<<dim3(H * bph, E), 128, smem, s>>>(b, cv, h->ld_cv, 0, nk, 2 * nk, h->f1 + c.b_heads, h->ld_f1, (const float*)L.A_log,
-                                             (const float*)L.dt_bias, H, G, dk, dv, bph, async_ok, L.rec_state, h->f2, h->ld_f2);
-  };
-  if (dk <= 16) launch(delta_head_kernel<AT, 16, 4>, 4, delta_head_smem<AT>(16, 4));
-  else if (dk <= 32) launch(delta_head_kernel<AT, 32, 4>, 4, delta_head_smem<AT>(32, 4));
-  else if (dk <= 64) launch(delta_head_kernel<AT, 64, 8>, 8, delta_head_smem<AT>(64, 8));
-  else if (dk <= 128) launch(delta_head_kernel<AT, 128, 16>, 16, delta_head_smem<AT>(128, 16));
-  else if (dk <= 256) launch(delta_head_kernel<AT, 256, 32>, 32, delta_head_smem<AT>(256, 32));
-  else if (dk <= 512) launch(delta_head_kernel<AT, 512, 32>, 32, delta_head_smem<AT>(512, 32));
-  else launch(delta_head_kernel<AT, 1024, 32>, 32, delta_head_smem<AT>(1024, 32));
+  launch_linear<AT>(dk, [&](auto dr, auto parts) {
+    constexpr int DR = decltype(dr)::value, PARTS = decltype(parts)::value;
+    const LinearLaunch g = linear_launch<AT>(PARTS, dk, dv, cv, h->ld_cv);
+    const size_t smem = lin_smem<AT>(DR, PARTS, 4);
+    cudaFuncSetAttribute(delta_head_kernel<AT, DR, PARTS>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    delta_head_kernel<AT, DR, PARTS><<<dim3(H * g.bph, E), 128, smem, s>>>(b, h->lin, cv, h->ld_cv, h->lin_sc, H, G, dk, dv, g.bph, g.vec, g.vvec,
+                                                                           L.rec_state, h->f2, h->ld_f2);
+  });
   gla_out_kernel<AT><<<(T * H + 3) / 4, 128, 0, s>>>(T, H, dv, h->f2, h->ld_f2, pin + L.c_g, h->ld_pin, L.g_norm, h->m.norm_eps,
                                                      c.right_scale, cat + L.o_scan, h->ld_cat);
   h->launches += 2;
