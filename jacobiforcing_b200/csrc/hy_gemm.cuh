@@ -18,13 +18,14 @@
 
 namespace hy {
 
-constexpr int TC_MAX_STAGES = 4;
-__host__ __device__ constexpr int tc_stages(int bt) { return 2; }   // three (two) blocks per SM: their prologues and epilogues overlap other blocks' products
+// Two stages: three blocks of 128 rows (two of 256) share an SM, and their prologues and epilogues run under the other blocks'
+// products; more stages in fewer blocks were slower at every size measured.
+constexpr int TC_STAGES = 2;
 constexpr int TC_WTILE = 128 * 64 * 2;                 // 16 KiB
 constexpr uint32_t TC_SPIN_LIMIT = 1u << 22;           // try_wait probes (each blocks for a bounded time itself)
 
 struct TcSmem {
-  uint64_t full[TC_MAX_STAGES], empty[TC_MAX_STAGES], acc_full;
+  uint64_t full[TC_STAGES], empty[TC_STAGES], acc_full;
   uint32_t tmem_base;
   uint32_t failed;
 };
@@ -53,7 +54,6 @@ __global__ void __launch_bounds__(192) gemm_tc_kernel(const bf16* __restrict__ X
                                                       int N, int K, GemmOut o, int* err, TcGroup grp) {
   extern __shared__ __align__(16) unsigned char hy_smem[];
   unsigned char* base = reinterpret_cast<unsigned char*>((reinterpret_cast<uintptr_t>(hy_smem) + 1023) & ~(uintptr_t)1023);
-  constexpr int TC_STAGES = tc_stages(BT);
   constexpr int XTILE = BT * 128;                        // BT rows of 64 bf16
   constexpr int SLOT = TC_WTILE + XTILE;
   TcSmem* sm = reinterpret_cast<TcSmem*>(base + TC_STAGES * SLOT);
@@ -178,7 +178,7 @@ __global__ void __launch_bounds__(192) gemm_tc_kernel(const bf16* __restrict__ X
   if (warp == 5) jf::tmem_dealloc(sm->tmem_base, BT);
 }
 
-constexpr size_t tc_smem_bytes(int bt) { return (size_t)tc_stages(bt) * (TC_WTILE + bt * 128) + sizeof(TcSmem) + 1024; }
+constexpr size_t tc_smem_bytes(int bt) { return (size_t)TC_STAGES * (TC_WTILE + bt * 128) + sizeof(TcSmem) + 1024; }
 
 // Host-side packer: row-major [N, K] floats -> bf16 tiles [ceil(N/128)][ceil(K/64)] of 128 x 64 in the swizzled layout.
 inline void pack_tiles(const float* w, int N, int K, std::vector<uint16_t>& out) {
