@@ -118,11 +118,59 @@ __global__ void __launch_bounds__(192) gemm_tc_kernel(const bf16* __restrict__ X
       const int pf = (o.act2 == 5 ? (n - lane - o.pair_lo) >> 1 : (n - lane) >> 1) + lane;      // this lane's feature of a pair
       const int pn = o.act2 == 5 ? o.pair_n : o.split, pld = o.act2 == 5 ? o.ld_pair : o.ld1;
       TO* pout = (TO*)(o.act2 == 5 ? o.pair_out : o.out1);
+      // what a column does with its elements is decided once: plain columns only scale and store (the general store's chain of
+      // tests per element cost more than the whole main loop at k = 1024)
+      const bool plain = !pairs && !o.resid && !o.bias && (o.act2 == 0 || o.act2 == 5);
+      const bool adds = o.resid && !o.post_w && !o.next_w && !o.bias;
+      const bool second = n >= o.split, wide = second ? (o.out2_f32 || sizeof(TO) == 4) : sizeof(TO) == 4;
+      const int pitch = second ? o.ld2 : o.ld1;
+      char* dst = second ? (char*)o.out2 + (size_t)(n - o.split) * (wide ? 4 : 2) : (char*)o.out1 + (size_t)n * sizeof(TO);
       for (int c0 = 0; c0 < BT; c0 += 16) {
         if (t0 + c0 >= T) break;
+        __syncwarp();                                        // the loads from tensor memory are warp-wide
         uint32_t v[16];
         jf::tmem_ld16(taddr + c0, v);
         jf::tmem_ld_wait();
+        const int rows = min(16, T - t0 - c0);
+        if (adds) {
+          if (n < N) {
+            float* p = o.resid + (size_t)(t0 + c0) * o.ldr + n;
+            float x[16];
+#pragma unroll
+            for (int j = 0; j < 16; ++j) x[j] = j < rows ? p[(size_t)j * o.ldr] : 0.0f;
+#pragma unroll
+            for (int j = 0; j < 16; ++j)
+              if (j < rows) p[(size_t)j * o.ldr] = fmaf(__uint_as_float(v[j]), o.alpha, x[j]);
+          }
+          continue;
+        }
+        if (plain) {
+          if (n >= N) {
+          } else if (wide) {
+            float* p = (float*)dst + (size_t)(t0 + c0) * pitch;
+#pragma unroll
+            for (int j = 0; j < 16; ++j)
+              if (j < rows) p[(size_t)j * pitch] = __uint_as_float(v[j]) * o.alpha;
+          } else {
+            bf16* p = (bf16*)dst + (size_t)(t0 + c0) * pitch;
+#pragma unroll
+            for (int j = 0; j < 16; ++j)
+              if (j < rows) p[(size_t)j * pitch] = __float2bfloat16_rn(__uint_as_float(v[j]) * o.alpha);
+          }
+          continue;
+        }
+        if (pairs && o.act_kind == 0) {                      // silu pairs: both halves of the warp work on 8 of the 16 tokens each
+#pragma unroll
+          for (int j = 0; j < 8; ++j) {
+            // lanes < 16 hold gates, the others ups: exchange so that a lane < 16 gets token j's pair and lane + 16 token j + 8's
+            const float give = __uint_as_float(lane < 16 ? v[j + 8] : v[j]);
+            const float got = __shfl_xor_sync(0xffffffffu, give, 16);
+            const float g = lane < 16 ? __uint_as_float(v[j]) : got, up = lane < 16 ? got : __uint_as_float(v[j + 8]);
+            const int row = lane < 16 ? j : j + 8, feat = pf - (lane & 16);
+            if (feat < pn && row < rows) pout[(size_t)(t0 + c0 + row) * pld + feat] = from_f<TO>(silu_f(g) * up);
+          }
+          continue;
+        }
         if (pairs) {
 #pragma unroll
           for (int j = 0; j < 16; ++j) {
